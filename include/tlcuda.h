@@ -59,7 +59,7 @@ enum {
  * stay quantized in device memory; Q6_K (210-byte super-blocks of 256 values) and
  * F32 are accepted on upload and become F16 tensors, which is what the reference's
  * loader makes of every type (src/model/formats/gguf.rs:128-253, :413-440). */
-enum { TLC_TYPE_F32 = 0, TLC_TYPE_F16 = 1, TLC_TYPE_Q4_0 = 2, TLC_TYPE_Q8_0 = 8, TLC_TYPE_Q6_K = 14 };
+enum { TLC_TYPE_F32 = 0, TLC_TYPE_F16 = 1, TLC_TYPE_Q4_0 = 2, TLC_TYPE_Q8_0 = 8, TLC_TYPE_Q6_K = 14, TLC_TYPE_BF16 = 30 };
 
 /* How a weight is split across tensor-parallel ranks. */
 enum {
@@ -237,6 +237,16 @@ TLC_API int32_t tlc_fill_normal_f16(tlc_ctx *ctx, void *dst_dev, size_t n, uint6
 TLC_API int32_t tlc_qtensor_create_normal_f16(tlc_ctx *ctx, int64_t n_rows, int64_t n_cols,
                                               uint64_t seed, uint64_t tensor_id, float mean,
                                               float std, tlc_qtensor **out);
+/* Dense weights of the models that do not come quantized: the host array `data` (row-major
+ * [n_rows, n_cols], src_type F32, F16 or BF16) is stored in HBM as store_type BF16 or F32, the
+ * latter kept in 32 bits (tlc_qtensor_create turns F32 into F16).  Rows start on 16-byte
+ * boundaries; the padding is zero. */
+TLC_API int32_t tlc_qtensor_create_dense(tlc_ctx *ctx, int32_t src_type, int32_t store_type, int64_t n_rows,
+                                         int64_t n_cols, const void *data, size_t bytes, tlc_qtensor **out);
+/* The same storage filled on the device with N(mean, std) draws of the counter-based generator. */
+TLC_API int32_t tlc_qtensor_create_normal_dense(tlc_ctx *ctx, int32_t store_type, int64_t n_rows, int64_t n_cols,
+                                                uint64_t seed, uint64_t tensor_id, float mean, float std,
+                                                tlc_qtensor **out);
 TLC_API int32_t tlc_qtensor_destroy(tlc_qtensor *qt);
 /* Local (per-rank) shape and storage.  For F16 tensors row_pitch is the
  * distance in bytes between rows in HBM (the row size rounded up to 16); for
@@ -356,6 +366,13 @@ typedef struct tlc_kvcache tlc_kvcache;
 TLC_API int32_t tlc_kvcache_create(tlc_ctx *ctx, int32_t n_layers, int32_t max_batch,
                                    int32_t max_seq, int32_t n_kv_heads, int32_t head_dim,
                                    tlc_kvcache **out);
+/* The same cache for models whose layers differ: layer l holds kv_heads[l] heads of head_dims[l]
+ * values, stored as `type` (TLC_TYPE_BF16 or TLC_TYPE_F32), every head's row padded with zeros to
+ * a multiple of 8 values; per layer K and V [max_batch, max_seq, kv_heads, padded dim].  The f16
+ * entry points below (append, attention) refuse such a cache. */
+TLC_API int32_t tlc_kvcache_create_layers(tlc_ctx *ctx, int32_t type, int32_t n_layers, int32_t max_batch,
+                                          int32_t max_seq, const int32_t *kv_heads, const int32_t *head_dims,
+                                          tlc_kvcache **out);
 TLC_API int32_t tlc_kvcache_destroy(tlc_kvcache *cache);
 TLC_API int32_t tlc_kvcache_layer_ptrs(tlc_kvcache *cache, int32_t layer, void **k_dev,
                                        void **v_dev);
@@ -428,6 +445,12 @@ TLC_API int32_t tlc_attention_decode_static_status(void *stream, int32_t *clampe
  * output: rows; attn_output/ffn_down: columns). */
 TLC_API int32_t tlc_model_load_gguf(tlc_ctx *ctx, const char *path, int32_t tp_rank,
                                     int32_t tp_size, tlc_model **out);
+/* A safetensors file (an 8-byte little-endian header length, a JSON header name -> dtype, shape,
+ * data_offsets, then the data): every tensor is uploaded with tlc_qtensor_create_dense as
+ * store_type (TLC_TYPE_BF16 or TLC_TYPE_F32); a tensor of rank 1 becomes [1, n], higher ranks
+ * keep the last dimension as columns.  Dtypes F32, F16 and BF16.  The shape, size and offsets of
+ * every tensor are checked against the file before anything is uploaded. */
+TLC_API int32_t tlc_model_load_safetensors(tlc_ctx *ctx, const char *path, int32_t store_type, tlc_model **out);
 /* Lazy weight cache: GGUFWeightCache (src/model/gguf_weight_cache.rs:45-262, :418-441;
  * builtins load_weight_cache_gguf_f16 / _f32 and get_weight, builtin_model.rs:330-414).
  * Opens the file and reads its tensor table; tlc_weight_cache_get uploads a tensor on
@@ -543,6 +566,70 @@ TLC_API int32_t tlc_temperature_sample(tlc_ctx *ctx, const void *logits_dev, int
  * gather + sampling); tokens and positions are left untouched unless parts == 7. */
 TLC_API int32_t tlc_llama_decode_enqueue_parts(tlc_llama *l, int32_t batch, int32_t steps,
                                                int32_t parts);
+/* ---- config-driven decoder ---------------------------------------------------- */
+
+/* A decoder-only transformer whose layers are described one by one: the mechanisms below, with
+ * their constants as parameters.  A layer adds its mixer, fed with one layer norm of the residual
+ * x, and its feed-forward, fed with another layer norm of the same x, to x; x is kept in 32 bits,
+ * weights and activations are BF16 or F32.
+ * Mixer: grouped-query attention.  Biases on q, k and the output; the projected keys double as the
+ * values; one RMS norm spans all query heads, one all key heads; then the first rot_dims entries
+ * of a head turn, entry e with entry e + rot_dims/2, by position * rot_base^(-2e/rot_dims).  Key j
+ * is visible to query i for 0 <= i - j < window, and for j <= i also when j < keep_first.
+ * Feed-forward (ff_kind):
+ *   TLC_FF_NONE          none;
+ *   TLC_FF_CLAMPED_GLU   down(g sigmoid(1.702 g) (u + 1)), g = min(gate, limit), u = up cut to +-limit;
+ *   TLC_FF_MOE           the `top` experts (silu(gate) * up) with the largest sigmoid scores, each fed
+ *                        with its score times the input; shared_ff > 0: one more expert for every
+ *                        token, times a sigmoid gate of its own.
+ * Logits: the embedding table against the final layer norm. */
+enum { TLC_FF_NONE = 0, TLC_FF_CLAMPED_GLU = 1, TLC_FF_MOE = 2 };
+typedef struct tlc_decoder_layer {
+    int32_t heads, kv_heads, dim;       /* query heads, key/value heads, size of a head     */
+    int32_t window, keep_first;         /* sliding window and the first tokens it keeps     */
+    int32_t rot_dims;
+    double rot_base;
+    float scale;                        /* of the scores                                    */
+    int32_t ff_kind, ff;                /* TLC_FF_*; ff: width of the dense feed-forward    */
+    float limit;
+    int32_t experts, top, expert_ff, shared_ff;
+} tlc_decoder_layer;
+typedef struct tlc_decoder_config {
+    int32_t n_layers, width, vocab;
+    float norm_eps;
+    int32_t dtype;           /* TLC_TYPE_BF16 or TLC_TYPE_F32: weights, activations, cache */
+    int32_t max_seq;         /* cache positions per sequence                               */
+    int32_t max_batch;       /* sequences held at once (<= 64)                             */
+    int32_t max_prefill;     /* rows one pass takes; longer portions run in several        */
+    int32_t max_logit_rows;  /* rows of logits one pass may be asked for                   */
+    int32_t no_graph;
+    const tlc_decoder_layer *layers;
+} tlc_decoder_config;
+typedef struct tlc_decoder tlc_decoder;
+/* Binds a model's tensors by name: "embed", "final.norm" and per layer "l<i>." + norm1, norm2,
+ * mix.{q,q.b,q.norm,k,k.b,k.norm,o,o.b}, mlp.{gate,up,down} or mlp.{router,e<j>.gate,e<j>.up,
+ * e<j>.down,shared.gate,shared.up,shared.down,shared.sg}. The model must outlive the decoder. */
+TLC_API int32_t tlc_decoder_create(tlc_ctx *ctx, tlc_model *model, const tlc_decoder_config *cfg, tlc_decoder **out);
+TLC_API int32_t tlc_decoder_destroy(tlc_decoder *d);
+/* The next n tokens of sequence `seq`, at positions pos0 .. pos0 + n - 1; pos0 must be where the
+ * sequence's earlier tokens end (smaller: it continues from there).  want[0..n_want): places among
+ * the n tokens, ascending, whose f32 logits [n_want, vocab] are written to logits_host.
+ * next_id_host: if not NULL the next token is sampled from the last row's logits, returned, and
+ * becomes the sequence's pending input. */
+TLC_API int32_t tlc_decoder_prefill(tlc_decoder *d, int32_t seq, const int32_t *ids_host, int32_t n, int32_t pos0,
+                                    const int32_t *want, int32_t n_want, float *logits_host, int32_t *next_id_host);
+/* Forgets sequence `seq`: its cache rows may be used again from position 0. */
+TLC_API int32_t tlc_decoder_release(tlc_decoder *d, int32_t seq);
+/* As the tlc_llama_* calls of the same names; logits are f32. */
+TLC_API int32_t tlc_decoder_set_state(tlc_decoder *d, int32_t batch, const int32_t *ids_host, const int32_t *positions_host);
+TLC_API int32_t tlc_decoder_decode_host(tlc_decoder *d, int32_t batch, const int32_t *ids_host, int32_t *next_ids_host,
+                                        float *logits_host);
+TLC_API int32_t tlc_decoder_decode_enqueue(tlc_decoder *d, int32_t batch, int32_t steps);
+TLC_API int32_t tlc_decoder_read_state(tlc_decoder *d, int32_t batch, int32_t *next_ids_host, int32_t *positions_host);
+TLC_API int32_t tlc_decoder_set_sampling(tlc_decoder *d, float temperature, uint64_t seed);
+TLC_API int32_t tlc_decoder_launches_per_step(tlc_decoder *d);
+TLC_API tlc_kvcache *tlc_decoder_cache(tlc_decoder *d);
+
 /* ---- tensor parallelism ----------------------------------------------------- */
 
 /* No counterpart in the reference (it has no multi-GPU code).  One process per

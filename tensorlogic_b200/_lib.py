@@ -17,7 +17,8 @@ ERR_SHAPE_MISMATCH, ERR_INVALID_OPERATION, ERR_DEVICE, ERR_CUDA = -1, -2, -3, -4
 ERR_ALLOCATION, ERR_LOAD, ERR_BUFFER_EXHAUSTED, ERR_INDEX = -5, -6, -7, -8
 ERR_INVALID_DIMENSION, ERR_TIMEOUT, ERR_COMM = -9, -10, -11
 
-TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0 = 0, 1, 2, 8
+TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0, TYPE_BF16 = 0, 1, 2, 8, 30
+FF_NONE, FF_CLAMPED_GLU, FF_MOE = 0, 1, 2
 SPLIT_NONE, SPLIT_ROWS, SPLIT_COLS = 0, 1, 2
 
 _ERROR_NAMES = {
@@ -48,6 +49,21 @@ class LlamaConfig(C.Structure):
                 ("rope_base", C.c_uint32), ("max_seq", C.c_int32), ("max_batch", C.c_int32),
                 ("max_prefill", C.c_int32), ("tp_rank", C.c_int32), ("tp_size", C.c_int32),
                 ("logits_all_rows", C.c_int32), ("no_graph", C.c_int32)]
+
+
+class DecoderLayer(C.Structure):
+    """tlc_decoder_layer of include/tlcuda.h."""
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("window", C.c_int32),
+                ("keep_first", C.c_int32), ("rot_dims", C.c_int32), ("rot_base", C.c_double), ("scale", C.c_float),
+                ("ff_kind", C.c_int32), ("ff", C.c_int32), ("limit", C.c_float), ("experts", C.c_int32),
+                ("top", C.c_int32), ("expert_ff", C.c_int32), ("shared_ff", C.c_int32)]
+
+
+class DecoderConfig(C.Structure):
+    """tlc_decoder_config of include/tlcuda.h."""
+    _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("norm_eps", C.c_float),
+                ("dtype", C.c_int32), ("max_seq", C.c_int32), ("max_batch", C.c_int32), ("max_prefill", C.c_int32),
+                ("max_logit_rows", C.c_int32), ("no_graph", C.c_int32), ("layers", C.POINTER(DecoderLayer))]
 
 
 vp, i32, i64, u32, u64, sz, f32 = C.c_void_p, C.c_int32, C.c_int64, C.c_uint32, C.c_uint64, C.c_size_t, C.c_float
@@ -83,6 +99,8 @@ PROTOTYPES = {
     "tlc_synth_blocks_host": (i32, [i32, u64, u64, i32, i64, i64, vp]),
     "tlc_fill_normal_f16": (i32, [vp, vp, sz, u64, u64, f32, f32]),
     "tlc_qtensor_create_normal_f16": (i32, [vp, i64, i64, u64, u64, f32, f32, P(vp)]),
+    "tlc_qtensor_create_dense": (i32, [vp, i32, i32, i64, i64, vp, sz, P(vp)]),
+    "tlc_qtensor_create_normal_dense": (i32, [vp, i32, i64, i64, u64, u64, f32, f32, P(vp)]),
     "tlc_qtensor_destroy": (i32, [vp]),
     "tlc_qtensor_info": (i32, [vp, P(i32), P(i64), P(i64), P(sz), P(vp)]),
     "tlc_qtensor_blocks": (i32, [vp, vp, vp]),
@@ -105,6 +123,7 @@ PROTOTYPES = {
     "tlc_swiglu_gate_up": (i32, [vp, vp, vp, vp, i32, vp, f32, vp]),
     "tlc_linear_residual": (i32, [vp, vp, vp, i32, vp, vp]),
     "tlc_kvcache_create": (i32, [vp, i32, i32, i32, i32, i32, P(vp)]),
+    "tlc_kvcache_create_layers": (i32, [vp, i32, i32, i32, i32, P(i32), P(i32), P(vp)]),
     "tlc_kvcache_destroy": (i32, [vp]),
     "tlc_kvcache_layer_ptrs": (i32, [vp, i32, P(vp), P(vp)]),
     "tlc_kvcache_append": (i32, [vp, vp, i32, vp, vp, i32, i32, vp]),
@@ -112,6 +131,7 @@ PROTOTYPES = {
     "tlc_attention_decode_static": (i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, i32, f32]),
     "tlc_attention_decode_static_status": (i32, [vp, vp]),
     "tlc_model_load_gguf": (i32, [vp, C.c_char_p, i32, i32, P(vp)]),
+    "tlc_model_load_safetensors": (i32, [vp, C.c_char_p, i32, P(vp)]),
     "tlc_gguf_open": (i32, [C.c_char_p, P(vp)]),
     "tlc_gguf_close": (i32, [vp]),
     "tlc_gguf_tensor_count": (i32, [vp]),
@@ -139,6 +159,17 @@ PROTOTYPES = {
     "tlc_llama_launches_per_step": (i32, [vp, i32]),
     "tlc_llama_cache": (vp, [vp]),
     "tlc_llama_set_sampling": (i32, [vp, f32, u64]),
+    "tlc_decoder_create": (i32, [vp, vp, P(DecoderConfig), P(vp)]),
+    "tlc_decoder_destroy": (i32, [vp]),
+    "tlc_decoder_prefill": (i32, [vp, i32, P(i32), i32, i32, P(i32), i32, P(f32), P(i32)]),
+    "tlc_decoder_release": (i32, [vp, i32]),
+    "tlc_decoder_set_state": (i32, [vp, i32, P(i32), P(i32)]),
+    "tlc_decoder_decode_host": (i32, [vp, i32, P(i32), P(i32), P(f32)]),
+    "tlc_decoder_decode_enqueue": (i32, [vp, i32, i32]),
+    "tlc_decoder_read_state": (i32, [vp, i32, P(i32), P(i32)]),
+    "tlc_decoder_set_sampling": (i32, [vp, f32, u64]),
+    "tlc_decoder_launches_per_step": (i32, [vp]),
+    "tlc_decoder_cache": (vp, [vp]),
     "tlc_sample_uniform_host": (f32, [u64, u32, u32]),
     "tlc_temperature_sample": (i32, [vp, vp, i32, i32, f32, P(f32), P(i32)]),
     "tlc_weight_cache_open": (i32, [vp, C.c_char_p, i64, P(vp)]),

@@ -5,6 +5,7 @@
 """
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -48,6 +49,12 @@ def _deps_mtime() -> float:
 
 def build(force: bool = False, verbose: bool = False, extra: list[str] | None = None) -> str:
     os.makedirs(OBJDIR, exist_ok=True)
+    with open(os.path.join(OBJDIR, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)  # two processes of a fresh checkout may ask at once
+        return _build(force, verbose, extra)
+
+
+def _build(force: bool, verbose: bool, extra: list[str] | None) -> str:
     nvcc = _nvcc()
     hdr_m = _deps_mtime()
     env = dict(os.environ)

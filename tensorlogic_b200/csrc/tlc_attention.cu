@@ -28,14 +28,6 @@
 
 #include "tlc_internal.h"
 
-struct tlc_kvcache {
-    tlc_ctx *ctx;
-    int n_layers, max_batch, max_seq, n_kv_heads, head_dim;
-    __half *k;  // [layer][batch][max_seq][n_kv_heads][head_dim]
-    __half *v;
-    size_t layer_stride;  // elements
-};
-
 namespace {
 
 constexpr int kTileKeys = 64;
@@ -713,6 +705,7 @@ int32_t tlc_launch_attention(tlc_ctx *ctx, tlc_kvcache *cache, int layer, const 
                              int batch, int I, int n_heads, int q_pos0, const int *positions_dev, int max_keys,
                              float scale, bool positions_settled) {
     TLC_REQUIRE(cache && q_dev && out_dev, TLC_ERR_INVALID_OPERATION, "attention: null pointer");
+    TLC_REQUIRE(cache->type == TLC_TYPE_F16, TLC_ERR_INVALID_OPERATION, "attention: the cache does not hold f16");
     TLC_REQUIRE(layer >= 0 && layer < cache->n_layers, TLC_ERR_INDEX, "Index out of bounds: index %d, size %d",
                 layer, cache->n_layers);
     TLC_REQUIRE(batch >= 1 && batch <= cache->max_batch, TLC_ERR_SHAPE_MISMATCH,
@@ -873,6 +866,23 @@ int32_t tlc_launch_attention(tlc_ctx *ctx, tlc_kvcache *cache, int layer, const 
     return TLC_OK;
 }
 
+// The two zero-filled arrays of a cache; frees `c` when they cannot be had.
+static int32_t kvcache_allocate(tlc_kvcache *c, size_t bytes) {
+    cudaError_t e = cudaMalloc(&c->k, bytes);
+    if (e == cudaSuccess) e = cudaMalloc(&c->v, bytes);
+    if (e == cudaSuccess) e = cudaMemsetAsync(c->k, 0, bytes, c->ctx->stream);
+    if (e == cudaSuccess) e = cudaMemsetAsync(c->v, 0, bytes, c->ctx->stream);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        if (c->k) cudaFree(c->k);
+        if (c->v) cudaFree(c->v);
+        delete c;
+        return tlc_fail(TLC_ERR_ALLOCATION, "KV cache allocation of 2 x %zu bytes failed: %s", bytes,
+                        cudaGetErrorString(e));
+    }
+    return TLC_OK;
+}
+
 extern "C" int32_t tlc_kvcache_create(tlc_ctx *ctx, int32_t n_layers, int32_t max_batch, int32_t max_seq,
                                       int32_t n_kv_heads, int32_t head_dim, tlc_kvcache **out) {
     if (int32_t rc = tlc_enter(ctx)) return rc;
@@ -882,25 +892,45 @@ extern "C" int32_t tlc_kvcache_create(tlc_ctx *ctx, int32_t n_layers, int32_t ma
                 TLC_ERR_INVALID_DIMENSION, "kvcache_create: bad shape");
     tlc_kvcache *c = new tlc_kvcache();
     c->ctx = ctx;
+    c->type = TLC_TYPE_F16;
+    c->elem = sizeof(__half);
     c->n_layers = n_layers;
     c->max_batch = max_batch;
     c->max_seq = max_seq;
     c->n_kv_heads = n_kv_heads;
     c->head_dim = head_dim;
     c->layer_stride = (size_t)max_batch * max_seq * n_kv_heads * head_dim;
-    const size_t bytes = c->layer_stride * n_layers * sizeof(__half);
-    cudaError_t e = cudaMalloc(&c->k, bytes);
-    if (e == cudaSuccess) e = cudaMalloc(&c->v, bytes);
-    if (e == cudaSuccess) e = cudaMemsetAsync(c->k, 0, bytes, ctx->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(c->v, 0, bytes, ctx->stream);
-    if (e != cudaSuccess) {
-        cudaGetLastError();
-        if (c->k) cudaFree(c->k);
-        if (c->v) cudaFree(c->v);
-        delete c;
-        return tlc_fail(TLC_ERR_ALLOCATION, "KV cache allocation of 2 x %zu bytes failed: %s", bytes,
-                        cudaGetErrorString(e));
+    for (int l = 0; l < n_layers; l++) c->layers.push_back({n_kv_heads, head_dim, head_dim, (size_t)l * c->layer_stride});
+    if (int32_t rc = kvcache_allocate(c, c->layer_stride * n_layers * c->elem)) return rc;
+    *out = c;
+    return TLC_OK;
+}
+
+extern "C" int32_t tlc_kvcache_create_layers(tlc_ctx *ctx, int32_t type, int32_t n_layers, int32_t max_batch,
+                                             int32_t max_seq, const int32_t *kv_heads, const int32_t *head_dims,
+                                             tlc_kvcache **out) {
+    if (int32_t rc = tlc_enter(ctx)) return rc;
+    TLC_REQUIRE(out && kv_heads && head_dims, TLC_ERR_INVALID_OPERATION, "kvcache_create_layers: null pointer");
+    *out = nullptr;
+    TLC_REQUIRE(type == TLC_TYPE_BF16 || type == TLC_TYPE_F32, TLC_ERR_INVALID_OPERATION,
+                "kvcache_create_layers: type %d (bf16 or f32)", type);
+    TLC_REQUIRE(n_layers > 0 && max_batch > 0 && max_seq > 0, TLC_ERR_INVALID_DIMENSION, "kvcache_create_layers: bad shape");
+    for (int l = 0; l < n_layers; l++)
+        TLC_REQUIRE(kv_heads[l] > 0 && head_dims[l] > 0, TLC_ERR_INVALID_DIMENSION, "kvcache_create_layers: bad layer %d", l);
+    tlc_kvcache *c = new tlc_kvcache();
+    c->ctx = ctx;
+    c->type = type;
+    c->elem = type == TLC_TYPE_F32 ? 4 : 2;
+    c->n_layers = n_layers;
+    c->max_batch = max_batch;
+    c->max_seq = max_seq;
+    size_t total = 0;
+    for (int l = 0; l < n_layers; l++) {
+        const int row = (head_dims[l] + 7) & ~7;
+        c->layers.push_back({kv_heads[l], head_dims[l], row, total});
+        total += (size_t)max_batch * max_seq * kv_heads[l] * row;
     }
+    if (int32_t rc = kvcache_allocate(c, total * c->elem)) return rc;
     *out = c;
     return TLC_OK;
 }
@@ -916,8 +946,9 @@ extern "C" int32_t tlc_kvcache_destroy(tlc_kvcache *cache) {
 
 extern "C" int32_t tlc_kvcache_layer_ptrs(tlc_kvcache *cache, int32_t layer, void **k_dev, void **v_dev) {
     TLC_REQUIRE(cache && layer >= 0 && layer < cache->n_layers, TLC_ERR_INDEX, "kvcache: bad layer %d", layer);
-    if (k_dev) *k_dev = cache->k + (size_t)layer * cache->layer_stride;
-    if (v_dev) *v_dev = cache->v + (size_t)layer * cache->layer_stride;
+    const size_t off = cache->layers[(size_t)layer].offset * cache->elem;
+    if (k_dev) *k_dev = reinterpret_cast<uint8_t *>(cache->k) + off;
+    if (v_dev) *v_dev = reinterpret_cast<uint8_t *>(cache->v) + off;
     return TLC_OK;
 }
 
@@ -926,6 +957,7 @@ extern "C" int32_t tlc_kvcache_append(tlc_ctx *ctx, tlc_kvcache *cache, int32_t 
                                       const int32_t *positions_dev) {
     if (int32_t rc = tlc_enter(ctx)) return rc;
     TLC_REQUIRE(cache && k_dev && v_dev, TLC_ERR_INVALID_OPERATION, "kvcache_append: null pointer");
+    TLC_REQUIRE(cache->type == TLC_TYPE_F16, TLC_ERR_INVALID_OPERATION, "kvcache_append: the cache does not hold f16");
     TLC_REQUIRE(layer >= 0 && layer < cache->n_layers, TLC_ERR_INDEX, "Index out of bounds: index %d, size %d",
                 layer, cache->n_layers);
     const bool batched = positions_dev != nullptr;

@@ -1,0 +1,252 @@
+// Row-wise steps of the config-driven decoder: embedding into the f32 residual stream, layer
+// norms, query/key norm + rotation + cache append, expert choice and the permutation of rows by
+// expert.
+#include "tlc_dense.cuh"
+
+namespace tlc_dense {
+
+namespace {
+
+template <typename T>
+__global__ void embed_rows_kernel(const T *__restrict__ table, int64_t pitch, int vocab, int d, const int *__restrict__ ids,
+                                  float *__restrict__ x) {
+    pdl_enter();  // ids are written by the previous step's sampling kernel
+    const int r = blockIdx.y;
+    int id = ids[r];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; never read outside
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < d; i += gridDim.x * blockDim.x)
+        x[(size_t)r * d + i] = to_f32(table[(size_t)id * pitch + i]);
+}
+
+// One CTA per row.
+template <typename T>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const NormParams p) {
+    extern __shared__ float row[];
+    __shared__ float red[33];
+    pdl_enter();
+    const int tid = threadIdx.x;
+    if (p.zero)
+        for (int i = blockIdx.x * blockDim.x + tid; i < p.n_zero; i += gridDim.x * blockDim.x) p.zero[i] = 0;
+    const int src = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+    float *x = p.x + (size_t)src * p.d;
+    float s = 0.f;
+    for (int i = tid; i < p.d; i += blockDim.x) {
+        float v = __ldcg(x + i);
+        if (p.y) {
+            float a = 0.f;
+            for (int t = 0; t < p.top; t++)
+                a += to_f32(static_cast<const T *>(p.y)[(size_t)p.place[(size_t)src * p.top + t] * p.y_pitch + i]);
+            v += a;
+            if (!p.rows) x[i] = v;
+        }
+        row[i] = v;
+        s += v;
+    }
+    const float mean = block_sum(s, red) / (float)p.d;
+    float q = 0.f;
+    for (int i = tid; i < p.d; i += blockDim.x) {
+        const float dlt = row[i] - mean;
+        q += dlt * dlt;
+    }
+    const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)p.d + p.eps);
+#pragma unroll
+    for (int o = 0; o < 2; o++) {
+        if (!p.w[o]) continue;
+        const T *w = static_cast<const T *>(p.w[o]);
+        T *out = static_cast<T *>(p.out[o]) + (size_t)blockIdx.x * p.ldo;
+        for (int i = tid; i < p.d; i += blockDim.x) out[i] = from_f32<T>((row[i] - mean) * rstd * to_f32(w[i]));
+    }
+}
+
+// One CTA per row: RMS norm of all query heads at once and of all key heads at once, rotation of
+// the first `rot` values of every head, queries to q_out, keys and raw keys (= values) to the cache.
+template <typename T>
+__global__ void __launch_bounds__(256) qk_rotate_kernel(const RotParams p) {
+    extern __shared__ float cs[];  // [rot / 2] cos, [rot / 2] sin
+    __shared__ float red[33];
+    pdl_enter();
+    const int tid = threadIdx.x, r = blockIdx.x;
+    const T *q = static_cast<const T *>(p.q) + (size_t)r * p.ldq, *k = static_cast<const T *>(p.k) + (size_t)r * p.ldk;
+    const int pos = p.pos[r], nq = p.H * p.D, nk = p.G * p.D, half = p.rot / 2;
+    float *sn = cs + half;
+    for (int i = tid; i < half; i += blockDim.x) sincosf((float)pos * p.freq[i], &sn[i], &cs[i]);
+    float s = 0.f;
+    for (int i = tid; i < nq; i += blockDim.x) {
+        const float v = to_f32(q[i]);
+        s += v * v;
+    }
+    const float rq = 1.0f / sqrtf(block_sum(s, red) / (float)nq + p.eps);
+    s = 0.f;
+    for (int i = tid; i < nk; i += blockDim.x) {
+        const float v = to_f32(k[i]);
+        s += v * v;
+    }
+    const float rk = 1.0f / sqrtf(block_sum(s, red) / (float)nk + p.eps);  // also a barrier behind cs / sn
+    auto value = [&](const T *src, const void *w, float scale, int head, int e) {
+        auto norm = [&](int at) { return to_f32(src[at]) * scale * to_f32(static_cast<const T *>(w)[at]); };
+        const int at = head * p.D + e;
+        if (e >= p.rot) return norm(at);
+        const float v = norm(at);
+        return e < half ? v * cs[e] - norm(at + half) * sn[e] : v * cs[e - half] + norm(at - half) * sn[e - half];
+    };
+    T *qo = static_cast<T *>(p.q_out) + (size_t)r * p.H * p.Dp;
+    for (int i = tid; i < p.H * p.Dp; i += blockDim.x) {
+        const int head = i / p.Dp, e = i - head * p.Dp;
+        qo[i] = from_f32<T>(e < p.D ? value(q, p.qn, rq, head, e) : 0.f);
+    }
+    if (pos < 0 || pos >= p.max_seq) {  // a cache row that does not exist: nothing is written, the host hears about it
+        if (tid == 0 && atomicCAS(&p.status->code, 0, TLC_DEV_INDEX) == 0) p.status->where = 401;
+        return;
+    }
+    const size_t base = ((size_t)p.slot[r] * p.max_seq + pos) * p.G * p.Dp;
+    T *kc = static_cast<T *>(p.kc) + base, *vc = static_cast<T *>(p.vc) + base;
+    for (int i = tid; i < p.G * p.Dp; i += blockDim.x) {
+        const int head = i / p.Dp, e = i - head * p.Dp;
+        kc[i] = from_f32<T>(e < p.D ? value(k, p.kn, rk, head, e) : 0.f);
+        vc[i] = e < p.D ? k[head * p.D + e] : from_f32<T>(0.f);
+    }
+}
+
+// One warp per token: the `top` largest sigmoid scores, the lowest index of equals first.
+__global__ void route_kernel(const RouteParams p) {
+    extern __shared__ float all[];
+    pdl_enter();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (r >= p.m) return;
+    float *score = all + (size_t)warp * p.experts;
+    for (int e = lane; e < p.experts; e += 32) score[e] = sigmoid_f(p.logits[(size_t)r * p.ld + e]);
+    __syncwarp();
+    for (int t = 0; t < p.top; t++) {
+        float best = -1.f;
+        int bi = p.experts;
+        for (int e = lane; e < p.experts; e += 32)
+            if (score[e] > best) {
+                best = score[e];
+                bi = e;
+            }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ov > best || (ov == best && oi < bi)) {
+                best = ov;
+                bi = oi;
+            }
+        }
+        if (bi >= p.experts) bi = 0;  // scores that are not numbers: stay inside the tables
+        if (lane == 0) {
+            score[bi] = -2.f;
+            p.chosen[(size_t)r * p.top + t] = bi;
+            p.weight[(size_t)r * p.top + t] = best;
+            p.rank[(size_t)r * p.top + t] = atomicAdd(p.count + bi, 1);
+        }
+        __syncwarp();
+    }
+}
+
+// Rows in the order of their experts: CTA r copies row r to its `top` places.
+template <typename T>
+__global__ void __launch_bounds__(256) permute_kernel(const PermuteParams p) {
+    extern __shared__ int start[];  // [experts + 1]
+    pdl_enter();
+    const int tid = threadIdx.x, r = blockIdx.x;
+    if (tid < 32) {  // exclusive sums of the experts' row counts, 32 at a time
+        int carry = 0;
+        for (int e0 = 0; e0 < p.experts; e0 += 32) {
+            const int e = e0 + tid;
+            const int c = e < p.experts ? p.count[e] : 0;
+            int incl = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int t = __shfl_up_sync(0xffffffffu, incl, o);
+                if (tid >= o) incl += t;
+            }
+            if (e < p.experts) start[e] = carry + incl - c;
+            carry += __shfl_sync(0xffffffffu, incl, 31);
+        }
+        if (tid == 0) start[p.experts] = carry;
+    }
+    __syncthreads();
+    if (r == 0)
+        for (int e = tid; e <= p.experts; e += blockDim.x) p.off[e] = start[e];
+    for (int t = 0; t < p.top; t++) {
+        const int at = r * p.top + t;
+        const int dst = start[p.chosen[at]] + p.rank[at];
+        if (tid == 0) {
+            p.place[at] = dst;
+            p.scale[dst] = p.weight[at];
+        }
+        // rows are whole 16-byte pieces (ldh is padded)
+        const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const T *>(p.h) + (size_t)r * p.ldh);
+        uint4 *to = reinterpret_cast<uint4 *>(static_cast<T *>(p.hp) + (size_t)dst * p.ldh);
+        for (int i = tid; i < p.ldh / Vec<T>::N; i += blockDim.x) to[i] = src[i];
+    }
+}
+
+}  // namespace
+
+#define TLC_LAUNCHED(ctx, le, what)                                                            \
+    do {                                                                                       \
+        if ((le) != cudaSuccess) {                                                             \
+            cudaGetLastError();                                                                \
+            return tlc_fail(TLC_ERR_CUDA, what " launch failed: %s", cudaGetErrorString(le));  \
+        }                                                                                      \
+        TLC_CHECK_LAUNCH(ctx);                                                                 \
+    } while (0)
+
+template <typename T>
+int32_t launch_embed(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int m, float *x) {
+    const int d = (int)table->n_cols, per = (d + 1023) / 1024;
+    cudaError_t le = tlc_launch_pdl(ctx, embed_rows_kernel<T>, dim3(per, m), dim3(256), 0, static_cast<const T *>(table->data),
+                                    (int64_t)(table->row_pitch / sizeof(T)), (int)table->n_rows, d, ids, x);
+    TLC_LAUNCHED(ctx, le, "embedding");
+    return TLC_OK;
+}
+
+template <typename T>
+int32_t launch_norm(tlc_ctx *ctx, const NormParams &p) {
+    const size_t smem = (size_t)p.d * sizeof(float);
+    static bool done[64] = {};
+    if (!done[ctx->device & 63]) {
+        TLC_CUDA(cudaFuncSetAttribute(norm_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        done[ctx->device & 63] = true;
+    }
+    TLC_REQUIRE(smem <= 200 * 1024, TLC_ERR_INVALID_OPERATION, "layer norm over %d values does not fit the shared memory", p.d);
+    cudaError_t le = tlc_launch_pdl(ctx, norm_rows_kernel<T>, dim3(p.m), dim3(256), smem, p);
+    TLC_LAUNCHED(ctx, le, "layer norm");
+    return TLC_OK;
+}
+
+template <typename T>
+int32_t launch_qk_rotate(tlc_ctx *ctx, const RotParams &p, int m) {
+    cudaError_t le = tlc_launch_pdl(ctx, qk_rotate_kernel<T>, dim3(m), dim3(256), (size_t)p.rot * sizeof(float) + 16, p);
+    TLC_LAUNCHED(ctx, le, "query/key norm");
+    return TLC_OK;
+}
+
+int32_t launch_route(tlc_ctx *ctx, const RouteParams &p) {
+    const int warps = p.experts > 1024 ? 1 : 8;
+    cudaError_t le = tlc_launch_pdl(ctx, route_kernel, dim3((p.m + warps - 1) / warps), dim3(32 * warps),
+                                    (size_t)warps * p.experts * sizeof(float), p);
+    TLC_LAUNCHED(ctx, le, "router");
+    return TLC_OK;
+}
+
+template <typename T>
+int32_t launch_permute(tlc_ctx *ctx, const PermuteParams &p) {
+    cudaError_t le = tlc_launch_pdl(ctx, permute_kernel<T>, dim3(p.m), dim3(256), ((size_t)p.experts + 1) * sizeof(int), p);
+    TLC_LAUNCHED(ctx, le, "expert permutation");
+    return TLC_OK;
+}
+
+template int32_t launch_embed<bf16>(tlc_ctx *, const tlc_qtensor *, const int *, int, float *);
+template int32_t launch_embed<float>(tlc_ctx *, const tlc_qtensor *, const int *, int, float *);
+template int32_t launch_norm<bf16>(tlc_ctx *, const NormParams &);
+template int32_t launch_norm<float>(tlc_ctx *, const NormParams &);
+template int32_t launch_qk_rotate<bf16>(tlc_ctx *, const RotParams &, int);
+template int32_t launch_qk_rotate<float>(tlc_ctx *, const RotParams &, int);
+template int32_t launch_permute<bf16>(tlc_ctx *, const PermuteParams &);
+template int32_t launch_permute<float>(tlc_ctx *, const PermuteParams &);
+
+}  // namespace tlc_dense

@@ -513,6 +513,8 @@ int32_t tlc_launch_gemv(tlc_ctx *ctx, const tlc_gemv_args &a) {
     const tlc_qtensor *w0 = a.outs[0].w;
     const int type = w0->type;
     const int64_t k = w0->n_cols;
+    TLC_REQUIRE(type != TLC_TYPE_BF16 && type != TLC_TYPE_F32, TLC_ERR_INVALID_OPERATION,
+                "linear: f16 activations need a quantized or f16 weight");
     for (int i = 0; i < a.n_out; i++) {
         const tlc_qtensor *w = a.outs[i].w;
         TLC_REQUIRE(w && a.outs[i].y, TLC_ERR_INVALID_OPERATION, "gemv: null weight or output");

@@ -119,6 +119,24 @@ struct tlc_qtensor {
     int32_t tp_rank, tp_size, split;
 };
 
+// One layer of a KV cache: K and V [max_batch][max_seq][heads][row] from element `offset` of the
+// cache's two arrays; row = head_dim padded to a multiple of 8 values (no padding in the f16 form).
+struct tlc_kvlayer {
+    int heads, dim, row;
+    size_t offset;
+};
+struct tlc_kvcache {
+    tlc_ctx *ctx;
+    int type;                             // TLC_TYPE_F16 (every layer alike), TLC_TYPE_BF16 or TLC_TYPE_F32
+    int n_layers, max_batch, max_seq;
+    int n_kv_heads, head_dim;             // f16 form
+    size_t elem;                          // bytes of a value
+    __half *k;                            // [layer][batch][max_seq][n_kv_heads][head_dim]
+    __half *v;
+    size_t layer_stride;                  // elements (f16 form)
+    std::vector<tlc_kvlayer> layers;
+};
+
 // ---- error plumbing -------------------------------------------------------
 int32_t tlc_fail(int32_t code, const char *fmt, ...);
 void tlc_clear_error();
@@ -262,7 +280,6 @@ int32_t tlc_gemv_splitk_finish(tlc_ctx *ctx, const tlc_gemv_args &a, int ksplit,
 // Scratch the fused GEMV may need for m rows (split-K partial sums; 0 when it does not split).
 size_t tlc_gemv_scratch_bytes(tlc_ctx *ctx, int type, int64_t k, int m, int64_t n_total);
 
-struct tlc_kvcache;
 int32_t tlc_launch_attention(tlc_ctx *ctx, tlc_kvcache *cache, int layer, const void *q_dev, void *out_dev,
                              int batch, int n_queries, int n_heads, int q_pos0, const int *positions_dev,
                              int max_keys, float scale, bool positions_settled);

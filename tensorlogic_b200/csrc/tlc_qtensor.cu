@@ -4,6 +4,8 @@
 //
 // Replaces the load-time CPU dequantization of the TensorLogic loaders
 // (src/model/formats/gguf.rs:22-112, :377-450; mmap_gguf.rs:383-439).
+#include <cuda_bf16.h>
+
 #include <cstring>
 
 #include "tlc_internal.h"
@@ -205,17 +207,18 @@ static size_t bytes_per_row(int32_t type, int64_t cols) {
     return (size_t)cols * 2;  // F16 (F32 is converted on the host first)
 }
 
+// `dense32`: an F32 tensor keeps its 32 bits (otherwise it becomes F16).
 static int32_t alloc_qtensor(tlc_ctx *ctx, int32_t type, int64_t rows, int64_t cols, int64_t full_rows,
                              int64_t full_cols, int32_t tp_rank, int32_t tp_size, int32_t split,
-                             tlc_qtensor **out) {
+                             tlc_qtensor **out, bool dense32 = false) {
     tlc_qtensor *qt = new tlc_qtensor();
     qt->ctx = ctx;
-    qt->type = type == TLC_TYPE_F32 ? TLC_TYPE_F16 : type;
+    qt->type = type == TLC_TYPE_F32 && !dense32 ? TLC_TYPE_F16 : type;
     qt->n_rows = rows;
     qt->n_cols = cols;
     qt->full_rows = full_rows;
     qt->full_cols = full_cols;
-    qt->row_bytes = bytes_per_row(qt->type, cols);
+    qt->row_bytes = qt->type == TLC_TYPE_F32 ? (size_t)cols * 4 : bytes_per_row(qt->type, cols);
     if (qt->type == TLC_TYPE_Q4_0 || qt->type == TLC_TYPE_Q8_0) {
         // Tiles of 16 rows; rows past N and blocks past K stay zero.
         qt->row_pitch = 0;
@@ -391,6 +394,118 @@ extern "C" int32_t tlc_qtensor_create(tlc_ctx *ctx, int32_t type, int64_t n_rows
     return TLC_OK;
 }
 
+namespace {
+
+inline float bf16_to_f32(uint16_t u) {
+    const uint32_t w = (uint32_t)u << 16;
+    float f;
+    memcpy(&f, &w, 4);
+    return f;
+}
+// f32 -> bf16, round to nearest even; a NaN stays one.
+inline uint16_t f32_to_bf16(float f) {
+    uint32_t w;
+    memcpy(&w, &f, 4);
+    if ((w & 0x7fffffffu) > 0x7f800000u) return (uint16_t)((w >> 16) | 0x40u);
+    return (uint16_t)((w + 0x7fffu + ((w >> 16) & 1u)) >> 16);
+}
+
+__global__ void fill_normal_dense_kernel(void *dst, int is_f32, int64_t rows, int64_t cols, int64_t pitch, uint64_t key,
+                                         float mean, float std) {
+    const int64_t n = rows * cols;
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+        const uint64_t r = tlc_mix64(key + (uint64_t)i);
+        const float u1 = ((float)(uint32_t)(r >> 40) + 1.0f) * (1.0f / 16777216.0f);
+        const float u2 = (float)(uint32_t)((r >> 16) & 0xffffffu) * (1.0f / 16777216.0f);
+        const float v = mean + std * sqrtf(-2.0f * logf(u1)) * cosf(6.2831853f * u2);
+        const int64_t at = (i / cols) * pitch + i % cols;
+        if (is_f32)
+            static_cast<float *>(dst)[at] = v;
+        else
+            static_cast<__nv_bfloat16 *>(dst)[at] = __float2bfloat16_rn(v);
+    }
+}
+
+int32_t alloc_dense(tlc_ctx *ctx, int32_t store_type, int64_t n_rows, int64_t n_cols, tlc_qtensor **out) {
+    TLC_REQUIRE(store_type == TLC_TYPE_BF16 || store_type == TLC_TYPE_F32, TLC_ERR_INVALID_OPERATION,
+                "dense tensors are stored as bf16 or f32 (type %d asked for)", store_type);
+    TLC_REQUIRE(n_rows > 0 && n_cols > 0, TLC_ERR_INVALID_DIMENSION, "dense tensor shape [%lld, %lld]", (long long)n_rows,
+                (long long)n_cols);
+    if (int32_t rc = alloc_qtensor(ctx, store_type, n_rows, n_cols, n_rows, n_cols, 0, 1, TLC_SPLIT_NONE, out, true)) return rc;
+    cudaError_t e = cudaMemsetAsync((*out)->data, 0, (*out)->bytes + 16, ctx->stream);  // the padding of the rows
+    if (e != cudaSuccess) {
+        tlc_qtensor_destroy(*out);
+        *out = nullptr;
+        return tlc_fail(TLC_ERR_CUDA, "weight upload failed: %s", cudaGetErrorString(e));
+    }
+    return TLC_OK;
+}
+
+}  // namespace
+
+extern "C" int32_t tlc_qtensor_create_dense(tlc_ctx *ctx, int32_t src_type, int32_t store_type, int64_t n_rows,
+                                            int64_t n_cols, const void *data, size_t bytes, tlc_qtensor **out) {
+    if (int32_t rc = tlc_enter(ctx)) return rc;
+    TLC_REQUIRE(out && data, TLC_ERR_INVALID_OPERATION, "qtensor_create_dense: null pointer");
+    *out = nullptr;
+    TLC_REQUIRE(src_type == TLC_TYPE_F32 || src_type == TLC_TYPE_F16 || src_type == TLC_TYPE_BF16, TLC_ERR_LOAD,
+                "dense tensors come as f32, f16 or bf16 (type %d given)", src_type);
+    tlc_qtensor *qt = nullptr;
+    if (int32_t rc = alloc_dense(ctx, store_type, n_rows, n_cols, &qt)) return rc;
+    const size_t n = (size_t)n_rows * (size_t)n_cols, src_elem = src_type == TLC_TYPE_F32 ? 4 : 2;
+    if (bytes < n * src_elem) {
+        tlc_qtensor_destroy(qt);
+        return tlc_fail(TLC_ERR_LOAD, "dense tensor [%lld, %lld] needs %zu bytes, got %zu", (long long)n_rows, (long long)n_cols,
+                        n * src_elem, bytes);
+    }
+    std::vector<uint8_t> conv;
+    const void *src = data;
+    if (src_type != store_type) {
+        conv.resize(n * (store_type == TLC_TYPE_F32 ? 4 : 2));
+        for (size_t i = 0; i < n; i++) {
+            const float v = src_type == TLC_TYPE_F32   ? static_cast<const float *>(data)[i]
+                            : src_type == TLC_TYPE_F16 ? __half2float(static_cast<const __half *>(data)[i])
+                                                       : bf16_to_f32(static_cast<const uint16_t *>(data)[i]);
+            if (store_type == TLC_TYPE_F32)
+                reinterpret_cast<float *>(conv.data())[i] = v;
+            else
+                reinterpret_cast<uint16_t *>(conv.data())[i] = f32_to_bf16(v);
+        }
+        src = conv.data();
+    }
+    cudaError_t e = cudaMemcpy2DAsync(qt->data, qt->row_pitch, src, qt->row_bytes, qt->row_bytes, (size_t)n_rows,
+                                      cudaMemcpyHostToDevice, ctx->stream);
+    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);  // `data` / `conv` may go away
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        tlc_qtensor_destroy(qt);
+        return tlc_fail(TLC_ERR_CUDA, "weight upload failed: %s", cudaGetErrorString(e));
+    }
+    *out = qt;
+    return TLC_OK;
+}
+
+extern "C" int32_t tlc_qtensor_create_normal_dense(tlc_ctx *ctx, int32_t store_type, int64_t n_rows, int64_t n_cols,
+                                                   uint64_t seed, uint64_t tensor_id, float mean, float std,
+                                                   tlc_qtensor **out) {
+    if (int32_t rc = tlc_enter(ctx)) return rc;
+    TLC_REQUIRE(out, TLC_ERR_INVALID_OPERATION, "qtensor_create_normal_dense: null pointer");
+    *out = nullptr;
+    tlc_qtensor *qt = nullptr;
+    if (int32_t rc = alloc_dense(ctx, store_type, n_rows, n_cols, &qt)) return rc;
+    const int is_f32 = store_type == TLC_TYPE_F32;
+    fill_normal_dense_kernel<<<4 * ctx->sm_count, 256, 0, ctx->stream>>>(qt->data, is_f32, n_rows, n_cols,
+                                                                        (int64_t)(qt->row_pitch / (is_f32 ? 4 : 2)),
+                                                                        tlc_synth_key(seed, tensor_id), mean, std);
+    ctx->launches++;
+    if (cudaGetLastError() != cudaSuccess) {
+        tlc_qtensor_destroy(qt);
+        return tlc_fail(TLC_ERR_CUDA, "weight fill failed");
+    }
+    *out = qt;
+    return TLC_OK;
+}
+
 extern "C" int32_t tlc_qtensor_create_synthetic(tlc_ctx *ctx, int32_t type, int64_t n_rows, int64_t n_cols,
                                                 uint64_t seed, uint64_t tensor_id, int32_t scale_log2,
                                                 int32_t tp_rank, int32_t tp_size, int32_t split,
@@ -535,6 +650,8 @@ extern "C" int32_t tlc_dequant(tlc_ctx *ctx, tlc_qtensor *qt, void *out_f16_dev)
     TLC_REQUIRE(qt && out_f16_dev, TLC_ERR_INVALID_OPERATION, "tlc_dequant: null pointer");
     TLC_REQUIRE(qt->ctx->device == ctx->device, TLC_ERR_DEVICE, "tlc_dequant: tensor lives on device %d, context on %d",
                 qt->ctx->device, ctx->device);
+    TLC_REQUIRE(qt->type != TLC_TYPE_BF16 && qt->type != TLC_TYPE_F32, TLC_ERR_INVALID_OPERATION,
+                "tlc_dequant: a dense bf16 / f32 tensor is not quantized");
     const int threads = 256;
     const uint8_t *data = static_cast<const uint8_t *>(qt->data);
     __half *out = static_cast<__half *>(out_f16_dev);

@@ -34,6 +34,22 @@ class LlamaArch:
     rms_eps: float = 1e-5
     rope_base: int = 10000
 
+    @classmethod
+    def from_model(cls, model: "Model") -> "LlamaArch":
+        """The configuration a GGUF file's ``llama.*`` metadata states (vocabulary: the embedding's rows)."""
+        def num(key, default=None):
+            v = model.meta("llama." + key)
+            if v is None:
+                if default is None:
+                    raise TensorError(_lib.ERR_LOAD, f"GGUF metadata has no 'llama.{key}'")
+                return default
+            return v
+        heads, width = int(num("attention.head_count")), int(num("embedding_length"))
+        return cls(int(num("block_count")), width, heads, int(num("attention.head_count_kv", heads)),
+                   int(num("attention.key_length", width // heads)), int(num("feed_forward_length")),
+                   model.get_tensor("token_embd.weight").shape[0], float(num("attention.layer_norm_rms_epsilon", 1e-5)),
+                   int(num("rope.freq_base", 10000)))
+
     def tensor_shapes(self) -> dict:
         """GGUF tensor names -> (rows, cols) in the loader's [out, in] order."""
         d, qd, kvd = self.d_model, self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim
