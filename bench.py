@@ -829,13 +829,118 @@ def run_prefill(args, rank: int, world: int, local: int) -> None:
     print(json.dumps(line), flush=True)
 
 
+def toposun_sizes() -> dict:
+    """name -> (decoder architecture, the LLaMA architecture with the same widths, heads and active feed-forward)."""
+    from tensorlogic_b200.decoder import DecoderArch, LayerArch
+    from tensorlogic_b200.model import LlamaArch
+
+    def dense(width, heads, kv, dim, ff, n):
+        l = LayerArch(heads, kv, dim, 1024, 4, dim // 2, 10000.0, dim ** -0.5, "clamped_glu", ff, 7.0)
+        return (DecoderArch(width, 32000, 1e-5, [l] * n), LlamaArch(n, width, heads, kv, dim, ff, 32000))
+
+    def experts(width, heads, kv, dim, n_exp, top, ff, shared, n):
+        l = LayerArch(heads, kv, dim, 1024, 4, dim // 2, 10000.0, dim ** -0.5, "moe", experts=n_exp, top=top, expert_ff=ff,
+                      shared_ff=shared)
+        return (DecoderArch(width, 32000, 1e-5, [l] * n), LlamaArch(n, width, heads, kv, dim, top * ff + shared, 32000))
+    return {"small": dense(2048, 32, 4, 64, 5632, 22), "wide": dense(4096, 32, 8, 128, 11008, 8),
+            "experts": experts(2048, 16, 4, 128, 64, 8, 1024, 2048, 8)}
+
+
+def run_toposun(args) -> None:
+    """--workload toposun --size small|wide|experts: Toposun at the sizes of a real model's layers (random
+    weights, bf16), prompt of 2048 tokens and greedy decode of one sequence behind it, beside the LLaMA
+    runner at the same widths with Q8_0 weights.  Prefill: whole calls from the ids on the host to the
+    sampled token back; decode: graph replays between two CUDA events.  Every step reads more weight
+    bytes than the L2 holds."""
+    import torch
+    from tensorlogic_b200 import synth
+    from tensorlogic_b200.api import Device
+    from tensorlogic_b200.decoder import Decoder, synthetic_decoder
+    from tensorlogic_b200.model import Llama, synthetic_model
+    tokens, K, W = 2048, args.steps, max(args.warmup, 3)
+    arch, twin = toposun_sizes()[args.size]
+    if args.layers:
+        arch.layers, twin.n_layers = arch.layers[:args.layers], min(args.layers, twin.n_layers)
+    KP = max(3, min(K, 20))
+    dev = Device(0)
+    peaks = load_peaks()
+    stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
+    ids = synth.token_ids(SEED, "toposun.prompt", tokens, arch.vocab)
+    max_seq = tokens + W + K + 16
+
+    def barrier():
+        dev.synchronize()
+        torch.cuda.synchronize()
+
+    def prefill_ms(runner):
+        for _ in range(W):
+            runner.prefill(ids, return_logits=False)
+        barrier()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        for _ in range(KP):
+            runner.prefill(ids, return_logits=False)
+        e1.record(stream)
+        barrier()
+        return e0.elapsed_time(e1) / KP
+
+    def measure(runner, weight_bytes, head_bytes, kv_bytes, params, clocks=None):
+        pre = prefill_ms(runner)
+        ms, launches = time_decode(dev, runner, stream, 1, K, W, barrier, clocks)
+        ms /= K
+        bytes_step = weight_bytes + head_bytes + kv_bytes
+        flops = 2.0 * params * tokens
+        return {"decode_tokens_per_s": 1e3 / ms, "decode_ms": ms, "decode_gb_per_s": bytes_step / ms / 1e6,
+                "decode_frac": bytes_step / ms / 1e6 / peaks["hbm_gbs"], "bytes_per_step": bytes_step,
+                "launches_per_step": launches / K, "prefill_tokens_per_s": tokens / pre * 1e3, "prefill_ms": pre,
+                "prefill_tflops": flops / pre / 1e9, "prefill_frac": flops / pre / 1e9 / peaks["bf16_tflops_sustained"]}
+
+    runner = Decoder(dev, synthetic_decoder(dev, arch, SEED), arch, max_seq=max_seq, max_prefill=tokens)
+    weights = sum(arch.layer_weight_bytes(l) for l in arch.layers)
+    kv = sum(2 * 2 * l.kv_heads * l.dim * min(tokens, l.window + l.keep_first) for l in arch.layers)
+    launches0 = dev.launch_count
+    with ClockSampler(0) as clocks:
+        ours = measure(runner, weights, arch.vocab * arch.width * 2, kv, weights // 2, clocks)
+    launches = dev.launch_count - launches0
+    clock_line = clocks.summary()
+    runner.prefill(ids, return_logits=False)
+    tok = [int(ids[0])]
+    n_e2e = min(K, 64)
+    t0 = time.perf_counter()
+    for _ in range(n_e2e):
+        tok = runner.decode(tok)[0]
+    e2e = n_e2e / (time.perf_counter() - t0)
+    closest = None
+    if not args.no_closest:
+        del runner
+        llm = Llama(dev, synthetic_model(dev, twin, SEED, qtype=8, device_embeddings=True), twin, max_seq=max_seq, max_prefill=tokens)
+        params = sum(r * c for n, (r, c) in twin.tensor_shapes().items() if n.startswith("blk.") and not n.endswith("norm.weight"))
+        closest = measure(llm, params // 32 * 34, twin.vocab * twin.d_model // 32 * 34,
+                          twin.n_layers * 2 * 2 * twin.n_kv_heads * twin.head_dim * tokens, params)
+        closest["model"] = "llama q8_0, same widths, heads and active feed-forward; full causal attention"
+    print(json.dumps({
+        "metric": "toposun_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": ours["decode_ms"], "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": f"toposun-{args.size}", "layers": len(arch.layers), "width": arch.width, "global_batch": 1,
+                   "seq_len": tokens, "window": 1024, "parallelism": "single",
+                   "l2": "the weights of a step exceed the 126 MB L2", "seed": SEED},
+        "e2e": {"value": e2e, "unit": "tokens/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4},
+        "gpu_launches": int(launches), "clocks": clock_line, "toposun": ours, "closest": closest,
+        "peaks": peaks}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "decode70b"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "decode70b", "toposun"],
                     help="decode: the headline workload (default); prefill: Llama-2-7B-shape 2048-token prefill; "
+                         "toposun: the Toposun decoder (--size) beside the LLaMA runner at equal widths; "
                          "decode70b: the Llama-2-70B-shape decode of the N > 1 runs on ONE GPU (the TP1 point)")
     ap.add_argument("--kernel", default=None, choices=["linear", "allreduce"],
                     help="micro-benchmark one kernel instead of the decode workload (see run_kernel)")
+    ap.add_argument("--size", default="small", choices=["small", "wide", "experts"], help="of --workload toposun")
+    ap.add_argument("--layers", type=int, default=0, help="--workload toposun: only the first so many layers (for profiles)")
+    ap.add_argument("--no-closest", action="store_true", help="--workload toposun: leave the LLaMA runner out")
     ap.add_argument("--qtype", default="q4_0", choices=["q4_0", "q8_0"])
     ap.add_argument("--n", type=int, default=28672)
     ap.add_argument("--k", type=int, default=8192)
@@ -860,6 +965,11 @@ def main() -> None:
         return
     if args.kernel == "linear":
         run_kernel(args)
+        return
+    if args.workload == "toposun":
+        if world > 1:
+            raise SystemExit("--workload toposun runs on one GPU")
+        run_toposun(args)
         return
     if world > 1:
         dist_setup(args.gpus)
