@@ -202,15 +202,21 @@ int32_t prepare(tlc_decoder *D) {
         rot_max = std::max<int64_t>(rot_max, (int64_t)c.heads * round8(c.dim));
         attn_max = std::max<int64_t>(attn_max, round8(c.heads * c.dim));
         act_max = std::max<int64_t>(act_max, round8(L.ff_width()));
-        int64_t in = c.heads * c.dim + L.ff_width() + 32;
+        ExpertParams ep{};
+        OutParams op{};
+        op.n = ep.k = w;
+        op.seg[op.n_seg++].k = c.heads * c.dim;
+        if (L.ff_width()) op.seg[op.n_seg++].k = L.ff_width();
         if (c.ff_kind == TLC_FF_MOE) {
             acte_max = std::max<int64_t>(acte_max, (int64_t)round8(c.expert_ff));
             experts_max = std::max<int64_t>(experts_max, c.experts);
             D->top_max = std::max(D->top_max, c.top);
-            in += (int64_t)c.top * round8(c.expert_ff);
-            if (c.top > 512) D->one_row_ok = false;
+            ep.experts = c.experts;
+            ep.top = op.top = c.top;
+            ep.ff = op.expert_k = c.expert_ff;
         }
-        if (!gemv_fits(w) || !out_gemv_fits(in)) D->one_row_ok = false;
+        const bool fits = cfg.dtype == TLC_TYPE_F32 ? layer_gemv_fits<float>(D->ctx, ep, op) : layer_gemv_fits<bf16>(D->ctx, ep, op);
+        if (!gemv_fits(w) || !fits) D->one_row_ok = false;
         if (c.rot_dims > 0) {
             std::vector<float> fr((size_t)c.rot_dims / 2);
             for (size_t i = 0; i < fr.size(); i++) fr[i] = (float)std::pow(c.rot_base, -2.0 * (double)i / (double)c.rot_dims);
@@ -441,9 +447,9 @@ int32_t layers_one_row(tlc_decoder *D, const Pass &ps) {
             if (int32_t rc = launch_expert_gemv<T>(ctx, e)) return rc;
         }
         OutParams o{};
-        o.seg[o.n_seg++] = {L.o->data, D->attn, (int)L.o->n_cols, (int)(L.o->row_pitch / es), 0, nullptr};
+        o.seg[o.n_seg++] = {L.o->data, D->attn, (int)L.o->n_cols, (int)(L.o->row_pitch / es), 0, 1, nullptr};
         if (L.down)
-            o.seg[o.n_seg++] = {L.down->data, D->act, (int)L.down->n_cols, (int)(L.down->row_pitch / es), 0,
+            o.seg[o.n_seg++] = {L.down->data, D->act, (int)L.down->n_cols, (int)(L.down->row_pitch / es), 0, 1,
                                 L.sg ? D->router_out + c.experts : nullptr};
         if (moe) {
             o.down = L.down_tab;
@@ -628,7 +634,8 @@ int32_t forward_t(tlc_decoder *D, const Pass &ps) {
     const int n = ps.want || ps.n_want ? ps.n_want : ps.m;
     if (n == 0) return TLC_OK;
     const bool single = n == 1 && gemv_fits(w);
-    const bool fused = single && pending < 0 && (ps.m == 1 || ps.want_single >= 0);
+    // the one-row kernel takes a residual row that starts on a 16-byte boundary
+    const bool fused = single && pending < 0 && (ps.m == 1 || (ps.want_single >= 0 && w % 4 == 0));
     if (!fused) {
         NormParams np{};
         np.x = D->x;

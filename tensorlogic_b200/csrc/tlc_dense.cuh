@@ -115,7 +115,7 @@ struct GemvParams {
     GemvSeg seg[6];
     int n_seg, v_total;   // virtual rows, even per segment
     int k, pitch;         // inputs; elements between weight rows
-    int ksplit_log2;      // warps sharing a row
+    int split;            // stretches a row is cut into
     int rows_cap;         // virtual rows of the busiest CTA (size of the partial-sum area)
     const float *x;       // f32 [k]: layer-normalized here with norm_w[input]
     const void *xn;       // T [k], used as it is when not null
@@ -136,7 +136,7 @@ struct ExpertParams {
     void *act;               // T [top][act_pitch]
     int *chosen;             // [top], written by CTA 0
     float *weight;           // [top]
-    int experts, top, k, pitch, ff, act_pitch, ksplit_log2, rows_cap;
+    int experts, top, k, pitch, ff, act_pitch, split, rows_cap;
 };
 template <typename T>
 int32_t launch_expert_gemv(tlc_ctx *ctx, ExpertParams &p);
@@ -146,6 +146,7 @@ struct OutSeg {
     const void *w;
     const void *in;       // T [k]
     int k, pitch, c0;     // c0: first 16-byte piece in the concatenation
+    int split;            // stretches a row is cut into
     const float *scale_logit;  // or null: the segment counts times sigmoid(*scale_logit)
 };
 struct OutParams {
@@ -158,14 +159,15 @@ struct OutParams {
     const void *bias;         // T [n] or null
     float *x;
     int n, pieces;            // 16-byte pieces of the whole concatenation
-    int ksplit_log2, rows_cap, prefetch;
+    int expert_split, rows_cap, prefetch;
 };
 template <typename T>
 int32_t launch_out_gemv(tlc_ctx *ctx, OutParams &p);
 
-// Can these run for a model with these sizes (shared memory of the inputs)?
+// Do the inputs of these launches fit the shared memory?  (Sizes only: pointers may be null.)
 bool gemv_fits(int k);
-bool out_gemv_fits(int64_t k_total);
+template <typename T>
+bool layer_gemv_fits(const tlc_ctx *ctx, ExpertParams e, OutParams o);
 
 // ---- many activation rows ------------------------------------------------------------------------
 struct GemmGroup {

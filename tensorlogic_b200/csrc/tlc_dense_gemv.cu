@@ -6,9 +6,10 @@
 //   expert_gemv_kernel  router decision, then gate/up of the chosen experts;
 //   out_gemv_kernel     the projections back into the residual stream -- attention output,
 //                       feed-forward down, chosen experts, shared expert -- as ONE sum per output.
-// All are bound by the weights' bytes.  A warp streams a weight row, or 1 / 2^s of one, in 16-byte
-// loads; CTAs own contiguous rows, the partial sums meet in shared memory after the last load, so
-// no barrier interrupts the stream.  The input sits in shared memory as f32, unrounded.
+// All are bound by the weights' bytes.  A warp streams stretches of weight rows in 16-byte loads that
+// roll on from one stretch to the next, so that a lane always has the same number in flight; CTAs own
+// contiguous rows, the partial sums meet in shared memory after the last load, so no barrier
+// interrupts the stream.  The input sits in shared memory as f32, unrounded.
 #include <cstring>
 
 #include "tlc_dense.cuh"
@@ -18,15 +19,57 @@ namespace tlc_dense {
 namespace {
 
 constexpr int kThreads = 512, kWarps = kThreads / 32;
-constexpr int kUnroll = 8;  // 16-byte loads in flight per lane
+constexpr int kBatch = 4;  // 16-byte loads of a lane per batch; two batches are in flight
 constexpr size_t kSmemMax = 200 * 1024;
 
 // Input layout in shared memory: piece c (16 bytes of weights) faces floats 4 c .. 4 c + 3 of plane
 // 0 and, for bf16, of plane 1, so that a warp's 16-byte reads fall on distinct banks.
+
+// Piece c of an input of `pieces`, as f32 in its places.
 template <typename T>
-__device__ __forceinline__ int plane_index(int i, int pieces) {
-    if (Vec<T>::N == 4) return i;
-    return (i >> 3) * 4 + (i & 3) + ((i >> 2) & 1) * pieces * 4;
+__device__ __forceinline__ void put_piece(float *in, int c, int pieces, const float (&f)[Vec<T>::N]) {
+    *reinterpret_cast<float4 *>(in + 4 * c) = make_float4(f[0], f[1], f[2], f[3]);
+    if constexpr (Vec<T>::N == 8) *reinterpret_cast<float4 *>(in + 4 * (pieces + c)) = make_float4(f[4], f[5], f[6], f[7]);
+}
+template <typename T>
+__device__ __forceinline__ void get_piece(const float *in, int c, int pieces, float (&f)[Vec<T>::N]) {
+    const float4 a = *reinterpret_cast<const float4 *>(in + 4 * c);
+    f[0] = a.x;
+    f[1] = a.y;
+    f[2] = a.z;
+    f[3] = a.w;
+    if constexpr (Vec<T>::N == 8) {
+        const float4 b = *reinterpret_cast<const float4 *>(in + 4 * (pieces + c));
+        f[4] = b.x;
+        f[5] = b.y;
+        f[6] = b.z;
+        f[7] = b.w;
+    }
+}
+// Piece c of n f32 values (rows start on 16-byte boundaries), zeros past n.
+template <typename T>
+__device__ __forceinline__ void load_f32_piece(const float *x, int c, int n, float (&f)[Vec<T>::N]) {
+    constexpr int N = Vec<T>::N;
+    if (N * c + N <= n) {
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+            const float4 v = __ldcg(reinterpret_cast<const float4 *>(x + N * c + j));
+            f[j] = v.x;
+            f[j + 1] = v.y;
+            f[j + 2] = v.z;
+            f[j + 3] = v.w;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; j++) f[j] = N * c + j < n ? __ldcg(x + N * c + j) : 0.f;
+    }
+}
+// Zeroes the values of piece c from n on.
+template <typename T>
+__device__ __forceinline__ void cut_piece(int c, int n, float (&f)[Vec<T>::N]) {
+#pragma unroll
+    for (int j = 0; j < Vec<T>::N; j++)
+        if (Vec<T>::N * c + j >= n) f[j] = 0.f;
 }
 
 __device__ __forceinline__ uint4 load_weight(const uint4 *p) {
@@ -59,42 +102,91 @@ __device__ __forceinline__ float dot_piece(const uint4 &w, const float *plane0, 
     return s;
 }
 
-// This lane's share of pieces [c_lo, c_hi) of a weight row against the input pieces of the same
-// numbers shifted by `shift`.
-template <typename T>
-__device__ __forceinline__ float dot_row(const uint4 *row, const float *plane0, const float *plane1, int c_lo, int c_hi,
-                                         int shift, int lane) {
-    float s = 0.f;
-    for (int c = c_lo + lane; c < c_hi; c += 32 * kUnroll) {
-        uint4 w[kUnroll];
+// A stretch of one weight row: pieces [lo, hi) of w against the input pieces of the same numbers
+// plus `shift`; its sum times `scale` goes to part[slot].
+struct Item {
+    const uint4 *w;
+    int lo, hi, shift, slot;
+    float scale;
+};
+
+// The items of a CTA: `rows` rows of `per_row` stretches each; warp w takes items w, w + kWarps, ...
+// in row order.  `item(row, stretch)` describes one.
+template <typename T, typename F>
+__device__ __forceinline__ void stream_items(int rows, int per_row, const float *plane0, const float *plane1, float *part, F item) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int dr = kWarps / per_row, dt = kWarps - dr * per_row;
+    struct Cursor {
+        int r, t;
+        Item it;
+    };
+    auto advance = [&](Cursor &c) {
+        c.r += dr;
+        c.t += dt;
+        if (c.t >= per_row) {
+            c.t -= per_row;
+            c.r++;
+        }
+        if (c.r < rows) c.it = item(c.r, c.t);
+    };
+    Cursor ld;
+    ld.r = warp / per_row;
+    ld.t = warp - ld.r * per_row;
+    if (ld.r >= rows) return;
+    ld.it = item(ld.r, ld.t);
+    Cursor use = ld;
+    float acc = 0.f;
+    auto load_batch = [&](uint4 (&w)[kBatch]) {
+        if (ld.r >= rows) return;
+        const uint4 *src = ld.it.w + ld.it.lo + lane;
+        const int left = ld.it.hi - ld.it.lo - lane;
 #pragma unroll
-        for (int u = 0; u < kUnroll; u++)
-            w[u] = c + 32 * u < c_hi ? load_weight(row + c + 32 * u) : make_uint4(0u, 0u, 0u, 0u);
+        for (int u = 0; u < kBatch; u++)
+            if (32 * u < left) w[u] = load_weight(src + 32 * u);
+        ld.it.lo += 32 * kBatch;
+        if (ld.it.lo >= ld.it.hi) advance(ld);
+    };
+    auto use_batch = [&](uint4 (&w)[kBatch]) {
+        const int c = use.it.lo + lane, left = use.it.hi - c;
 #pragma unroll
-        for (int u = 0; u < kUnroll; u++)
-            if (c + 32 * u < c_hi) s += dot_piece<T>(w[u], plane0, plane1, c + 32 * u + shift);
+        for (int u = 0; u < kBatch; u++)
+            if (32 * u < left) acc += dot_piece<T>(w[u], plane0, plane1, c + 32 * u + use.it.shift);
+        use.it.lo += 32 * kBatch;
+        if (use.it.lo >= use.it.hi) {
+            acc = warp_sum(acc);
+            if (lane == 0) part[use.it.slot] = acc * use.it.scale;
+            acc = 0.f;
+            advance(use);
+        }
+    };
+    uint4 a[kBatch], b[kBatch];
+    load_batch(a);
+    while (use.r < rows) {
+        load_batch(b);
+        use_batch(a);
+        if (use.r >= rows) break;
+        load_batch(a);
+        use_batch(b);
     }
-    return s;
 }
 
-struct Share {  // pieces of a row warp `part` of 2^log2 takes
-    int lo, hi;
-};
-__device__ __forceinline__ Share share_of(int pieces, int part, int log2) {
-    const int per = (pieces + (1 << log2) - 1) >> log2;
+// Stretch `part` of a row of `pieces` cut every `per` pieces.
+__device__ __forceinline__ void share_of(int per, int pieces, int part, Item &it) {
     const int lo = part * per;
-    return {lo < pieces ? lo : pieces, lo + per < pieces ? lo + per : pieces};
+    it.lo = lo < pieces ? lo : pieces;
+    it.hi = lo + per < pieces ? lo + per : pieces;
 }
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const __grid_constant__ GemvParams p) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[33];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x;
     const int pieces = (p.k + Vec<T>::N - 1) / Vec<T>::N;
     const int row_floats = pieces * Vec<T>::N;
     float *xs[2] = {smem, smem + row_floats};
-    float *part = smem + 2 * (size_t)row_floats;
+    uint4 *nw = reinterpret_cast<uint4 *>(smem + 2 * (size_t)row_floats);  // the two norm weights, [2][pieces]
+    float *part = reinterpret_cast<float *>(nw + (p.xn ? 0 : 2 * pieces));
 
     // virtual rows of this CTA, cut at even numbers
     const int pairs = p.v_total >> 1;
@@ -118,62 +210,81 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const __grid_constant
         const T *w = weight_row(find(v_lo + tid), v_lo + tid);
         if (w) prefetch_l2(w, (uint32_t)(row_floats * sizeof(T)));
     }
-    bool need[2] = {false, p.h_out != nullptr && blockIdx.x == 0};
+    int need = p.h_out && blockIdx.x == 0 ? 2 : 0;  // bit i: this CTA's rows read normalized input i
     if (v_lo < v_hi)
-        for (int s = find(v_lo); s < p.n_seg && p.seg[s].v0 < v_hi; s++) need[p.seg[s].input] = true;
+        for (int s = find(v_lo); s < p.n_seg && p.seg[s].v0 < v_hi; s++) need |= 1 << p.seg[s].input;
+    if (!p.xn)
+#pragma unroll 4
+        for (int c = tid; c < 2 * pieces; c += kThreads) {
+            const int o = c >= pieces;
+            if (need >> o & 1) nw[c] = __ldg(static_cast<const uint4 *>(p.norm_w[o]) + (c - o * pieces));
+        }
     pdl_enter();
 
+    constexpr int N = Vec<T>::N;
     if (p.xn) {
-        const T *x = static_cast<const T *>(p.xn);
-        for (int i = tid; i < row_floats; i += kThreads) xs[0][plane_index<T>(i, pieces)] = i < p.k ? to_f32(x[i]) : 0.f;
+#pragma unroll 4
+        for (int c = tid; c < pieces; c += kThreads) {
+            float f[N];
+            unpack(__ldcg(static_cast<const uint4 *>(p.xn) + c), f);
+            cut_piece<T>(c, p.k, f);
+            put_piece<T>(xs[0], c, pieces, f);
+        }
     } else {
         float s = 0.f;
-        for (int i = tid; i < row_floats; i += kThreads) {
-            const float v = i < p.k ? __ldcg(p.x + i) : 0.f;
-            xs[1][plane_index<T>(i, pieces)] = v;
-            s += v;
+#pragma unroll 2
+        for (int c = tid; c < pieces; c += kThreads) {
+            float f[N];
+            load_f32_piece<T>(p.x, c, p.k, f);
+            put_piece<T>(xs[1], c, pieces, f);
+#pragma unroll
+            for (int j = 0; j < N; j++) s += f[j];
         }
         const float mean = block_sum(s, red) / (float)p.k;
         float q = 0.f;
-        for (int i = tid; i < p.k; i += kThreads) {
-            const float dlt = xs[1][plane_index<T>(i, pieces)] - mean;
-            q += dlt * dlt;
+        for (int c = tid; c < pieces; c += kThreads) {
+            float f[N];
+            get_piece<T>(xs[1], c, pieces, f);
+#pragma unroll
+            for (int j = 0; j < N; j++) q += N * c + j < p.k ? (f[j] - mean) * (f[j] - mean) : 0.f;
         }
         const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)p.k + p.eps);
-        const T *w0 = static_cast<const T *>(p.norm_w[0]), *w1 = static_cast<const T *>(p.norm_w[1]);
-        for (int i = tid; i < p.k; i += kThreads) {
-            const int at = plane_index<T>(i, pieces);
-            const float xh = (xs[1][at] - mean) * rstd;
-            if (need[0]) xs[0][at] = xh * to_f32(w0[i]);
-            if (need[1]) {
-                const float h = xh * to_f32(w1[i]);
-                xs[1][at] = h;
-                if (p.h_out && blockIdx.x == 0) p.h_out[i] = h;
+        for (int c = tid; c < pieces; c += kThreads) {
+            float f[N], w[N], h[N];
+            get_piece<T>(xs[1], c, pieces, f);
+#pragma unroll
+            for (int o = 0; o < 2; o++) {
+                if (!(need >> o & 1)) continue;
+                unpack(nw[o * pieces + c], w);  // padded with zeros
+#pragma unroll
+                for (int j = 0; j < N; j++) h[j] = (f[j] - mean) * rstd * w[j];
+                put_piece<T>(xs[o], c, pieces, h);
             }
+            if (p.h_out && blockIdx.x == 0)
+#pragma unroll
+                for (int j = 0; j < N; j++)
+                    if (N * c + j < p.k) p.h_out[N * c + j] = h[j];
         }
-        if (need[0])
-            for (int i = p.k + tid; i < row_floats; i += kThreads) xs[0][plane_index<T>(i, pieces)] = 0.f;
     }
     __syncthreads();
 
-    const int rows = v_hi - v_lo, ks = 1 << p.ksplit_log2;
-    for (int it = warp; it < rows << p.ksplit_log2; it += kWarps) {
-        const int r = it >> p.ksplit_log2, pt = it & (ks - 1);
+    const int rows = v_hi - v_lo, per = (pieces + p.split - 1) / p.split;
+    stream_items<T>(rows, p.split, smem, smem + 4 * pieces, part, [&](int r, int t) {
+        Item it;
         const int s = find(v_lo + r);
         const T *w = weight_row(s, v_lo + r);
-        float acc = 0.f;
-        if (w) {
-            const Share sh = share_of(pieces, pt, p.ksplit_log2);
-            const float *in = xs[p.seg[s].input];
-            acc = dot_row<T>(reinterpret_cast<const uint4 *>(w), in, in + 4 * pieces, sh.lo, sh.hi, 0, lane);
-            acc = warp_sum(acc);
-        }
-        if (lane == 0) part[it] = acc;
-    }
+        share_of(per, pieces, t, it);
+        if (!w) it.hi = it.lo;
+        it.w = reinterpret_cast<const uint4 *>(w);
+        it.shift = p.seg[s].input ? pieces * (Vec<T>::N / 4) : 0;  // the second input lies behind the first
+        it.slot = r * p.split + t;
+        it.scale = 1.f;
+        return it;
+    });
     __syncthreads();
     auto total = [&](int r) {
         float a = 0.f;
-        for (int i = 0; i < ks; i++) a += part[(r << p.ksplit_log2) + i];
+        for (int i = 0; i < p.split; i++) a += part[r * p.split + i];
         return a;
     };
     for (int r = tid; r < rows; r += kThreads) {
@@ -234,20 +345,32 @@ __device__ __forceinline__ void choose_experts(const float *logits, int experts,
 // writer of everything read here -- is complete.  It waits for the attention only before it ends,
 // so that whoever waits for this kernel has waited for both.
 template <typename T>
-__global__ void __launch_bounds__(kThreads, 2) expert_gemv_kernel(const __grid_constant__ ExpertParams p, int wait_first) {
+__global__ void __launch_bounds__(kThreads, 2) expert_gemv_kernel(const __grid_constant__ ExpertParams p) {
     extern __shared__ __align__(16) float smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int pieces = (p.k + Vec<T>::N - 1) / Vec<T>::N;
     const int row_floats = pieces * Vec<T>::N;
     float *xs = smem, *part = smem + row_floats;
-    float *score = part + ((size_t)p.rows_cap << p.ksplit_log2);
+    float *score = part + (size_t)p.rows_cap * p.split;
     float *weight = score + p.experts;
     int *chosen = reinterpret_cast<int *>(weight + p.top);
-    if (wait_first) pdl_wait();
+    const void **tab = reinterpret_cast<const void **>((reinterpret_cast<uintptr_t>(chosen + p.top) + 7) & ~(uintptr_t)7);  // [top][gate, up]
     pdl_trigger();
 
-    if (warp == 0) choose_experts(p.logits, p.experts, p.top, score, chosen, weight, lane);
-    for (int i = tid; i < row_floats; i += kThreads) xs[plane_index<T>(i, pieces)] = i < p.k ? __ldcg(p.h + i) : 0.f;
+    if (warp == 0) {
+        choose_experts(p.logits, p.experts, p.top, score, chosen, weight, lane);
+        for (int t = lane; t < p.top; t += 32) {
+            tab[2 * t] = p.gate[chosen[t]];
+            tab[2 * t + 1] = p.up[chosen[t]];
+        }
+    } else {
+#pragma unroll 2
+        for (int c = tid - 32; c < pieces; c += kThreads - 32) {
+            float f[Vec<T>::N];
+            load_f32_piece<T>(p.h, c, p.k, f);
+            put_piece<T>(xs, c, pieces, f);
+        }
+    }
     __syncthreads();
     if (blockIdx.x == 0 && tid < p.top) {
         p.chosen[tid] = chosen[tid];
@@ -257,35 +380,38 @@ __global__ void __launch_bounds__(kThreads, 2) expert_gemv_kernel(const __grid_c
     const int pairs = p.top * p.ff;
     const int u_lo = (int)((long long)pairs * blockIdx.x / gridDim.x);
     const int u_hi = (int)((long long)pairs * (blockIdx.x + 1) / gridDim.x);
-    const int rows = 2 * (u_hi - u_lo), ks = 1 << p.ksplit_log2;
-    for (int it = warp; it < rows << p.ksplit_log2; it += kWarps) {
-        const int r = it >> p.ksplit_log2, pt = it & (ks - 1);
-        const int u = u_lo + (r >> 1), c = u / p.ff, j = u - c * p.ff;
-        const void *w = r & 1 ? p.up[chosen[c]] : p.gate[chosen[c]];
-        const Share sh = share_of(pieces, pt, p.ksplit_log2);
-        float acc = dot_row<T>(reinterpret_cast<const uint4 *>(static_cast<const T *>(w) + (size_t)j * p.pitch), xs,
-                               xs + 4 * pieces, sh.lo, sh.hi, 0, lane);
-        acc = warp_sum(acc);
-        if (lane == 0) part[it] = acc;
-    }
+    const int per = (pieces + p.split - 1) / p.split;
+    stream_items<T>(2 * (u_hi - u_lo), p.split, xs, xs + 4 * pieces, part, [&](int r, int t) {
+        Item it;
+        const int u = u_lo + (r >> 1), c = u / p.ff;
+        const void *w = tab[2 * c + (r & 1)];
+        share_of(per, pieces, t, it);
+        it.w = reinterpret_cast<const uint4 *>(static_cast<const T *>(w) + (size_t)(u - c * p.ff) * p.pitch);
+        it.shift = 0;
+        it.slot = r * p.split + t;
+        it.scale = 1.f;
+        return it;
+    });
     __syncthreads();
     for (int u = u_lo + tid; u < u_hi; u += kThreads) {
         const int c = u / p.ff, j = u - c * p.ff, r = 2 * (u - u_lo);
         float gate = 0.f, up = 0.f;
-        for (int i = 0; i < ks; i++) {
-            gate += part[(r << p.ksplit_log2) + i];
-            up += part[((r + 1) << p.ksplit_log2) + i];
+        for (int i = 0; i < p.split; i++) {
+            gate += part[r * p.split + i];
+            up += part[(r + 1) * p.split + i];
         }
         static_cast<T *>(p.act)[(size_t)c * p.act_pitch + j] = from_f32<T>(silu_mul(weight[c] * gate, weight[c] * up));
     }
-    if (!wait_first) pdl_wait();
+    pdl_wait();
 }
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads, 2) out_gemv_kernel(const __grid_constant__ OutParams p) {
     extern __shared__ __align__(16) float smem[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x;
     float *part = smem + (size_t)p.pieces * Vec<T>::N;
+    const int slots = p.seg[0].split + (p.n_seg > 1 ? p.seg[1].split : 0) + p.top * p.expert_split;
+    const void **down = reinterpret_cast<const void **>(part + (((size_t)p.rows_cap * slots + 1) & ~(size_t)1));
     const int r_lo = (int)((long long)p.n * blockIdx.x / gridDim.x);
     const int r_hi = (int)((long long)p.n * (blockIdx.x + 1) / gridDim.x);
     for (int s = 0; s < p.n_seg; s++)
@@ -293,86 +419,102 @@ __global__ void __launch_bounds__(kThreads, 2) out_gemv_kernel(const __grid_cons
             prefetch_l2(static_cast<const T *>(p.seg[s].w) + (size_t)(r_lo + tid) * p.seg[s].pitch,
                         (uint32_t)(((p.seg[s].k * (int)sizeof(T)) + 15) & ~15));
     pdl_enter();
+    const int n_dense = p.expert_c0;
+#pragma unroll 4
+    for (int c = tid; c < p.pieces; c += kThreads) {
+        const T *in;
+        int at, k;
+        if (c < n_dense) {
+            const int s = p.n_seg > 1 && c >= p.seg[1].c0 ? 1 : 0;
+            in = static_cast<const T *>(p.seg[s].in);
+            at = c - p.seg[s].c0;
+            k = p.seg[s].k;
+        } else {
+            const int e = (c - n_dense) / p.expert_pieces;
+            in = static_cast<const T *>(p.expert_in) + (size_t)e * p.expert_in_pitch;
+            at = c - n_dense - e * p.expert_pieces;
+            k = p.expert_k;
+        }
+        float f[Vec<T>::N];
+        unpack(__ldcg(reinterpret_cast<const uint4 *>(in) + at), f);
+        cut_piece<T>(at, k, f);
+        put_piece<T>(smem, c, p.pieces, f);
+    }
     float seg_scale[2] = {1.f, 1.f};
-    for (int s = 0; s < p.n_seg; s++) {
-        const T *in = static_cast<const T *>(p.seg[s].in);
-        const int n = (p.seg[s].k + Vec<T>::N - 1) / Vec<T>::N * Vec<T>::N, base = p.seg[s].c0 * Vec<T>::N;
-        for (int i = tid; i < n; i += kThreads)
-            smem[plane_index<T>(base + i, p.pieces)] = i < p.seg[s].k ? to_f32(__ldcg(in + i)) : 0.f;
+    for (int s = 0; s < p.n_seg; s++)
         if (p.seg[s].scale_logit) seg_scale[s] = sigmoid_f(__ldcg(p.seg[s].scale_logit));
-    }
-    for (int c = 0; c < p.top; c++) {
-        const T *in = static_cast<const T *>(p.expert_in) + (size_t)c * p.expert_in_pitch;
-        const int n = p.expert_pieces * Vec<T>::N, base = (p.expert_c0 + c * p.expert_pieces) * Vec<T>::N;
-        for (int i = tid; i < n; i += kThreads)
-            smem[plane_index<T>(base + i, p.pieces)] = i < p.expert_k ? to_f32(__ldcg(in + i)) : 0.f;
-    }
+    if (tid < p.top) down[tid] = p.down[__ldcg(p.chosen + tid)];
     __syncthreads();
-    const float *plane1 = smem + 4 * (size_t)p.pieces;
-    const int rows = r_hi - r_lo, ks = 1 << p.ksplit_log2;
-    for (int it = warp; it < rows << p.ksplit_log2; it += kWarps) {
-        const int n = r_lo + (it >> p.ksplit_log2);
-        const Share sh = share_of(p.pieces, it & (ks - 1), p.ksplit_log2);
-        float acc = 0.f;
-        for (int s = 0; s < p.n_seg; s++) {
-            const int c0 = p.seg[s].c0, c1 = c0 + (p.seg[s].k + Vec<T>::N - 1) / Vec<T>::N;
-            const int lo = sh.lo > c0 ? sh.lo : c0, hi = sh.hi < c1 ? sh.hi : c1;
-            if (lo >= hi) continue;
-            acc += seg_scale[s] * dot_row<T>(reinterpret_cast<const uint4 *>(static_cast<const T *>(p.seg[s].w) +
-                                                                             (size_t)n * p.seg[s].pitch),
-                                             smem, plane1, lo - c0, hi - c0, c0, lane);
+    const int rows = r_hi - r_lo;
+    const int split0 = p.seg[0].split, split1 = p.n_seg > 1 ? p.seg[1].split : 0;
+    const int pieces0 = (p.seg[0].k + Vec<T>::N - 1) / Vec<T>::N, per0 = (pieces0 + split0 - 1) / split0;
+    const int pieces1 = split1 ? (p.seg[1].k + Vec<T>::N - 1) / Vec<T>::N : 0, per1 = split1 ? (pieces1 + split1 - 1) / split1 : 1;
+    const int per_e = (p.expert_pieces + p.expert_split - 1) / p.expert_split;
+    stream_items<T>(rows, slots, smem, smem + 4 * (size_t)p.pieces, part, [&](int r, int t) {
+        Item it;
+        it.slot = r * slots + t;
+        it.scale = 1.f;
+        if (t < split0) {
+            share_of(per0, pieces0, t, it);
+            it.w = reinterpret_cast<const uint4 *>(static_cast<const T *>(p.seg[0].w) + (size_t)(r_lo + r) * p.seg[0].pitch);
+            it.shift = 0;
+            it.scale = seg_scale[0];
+        } else if (t < split0 + split1) {
+            share_of(per1, pieces1, t - split0, it);
+            it.w = reinterpret_cast<const uint4 *>(static_cast<const T *>(p.seg[1].w) + (size_t)(r_lo + r) * p.seg[1].pitch);
+            it.shift = p.seg[1].c0;
+            it.scale = seg_scale[1];
+        } else {
+            t -= split0 + split1;
+            const int c = p.expert_split == 1 ? t : t / p.expert_split;
+            share_of(per_e, p.expert_pieces, t - c * p.expert_split, it);
+            it.w = reinterpret_cast<const uint4 *>(static_cast<const T *>(down[c]) + (size_t)(r_lo + r) * p.expert_pitch);
+            it.shift = p.expert_c0 + c * p.expert_pieces;
         }
-        for (int c = 0; c < p.top; c++) {
-            const int c0 = p.expert_c0 + c * p.expert_pieces, c1 = c0 + p.expert_pieces;
-            const int lo = sh.lo > c0 ? sh.lo : c0, hi = sh.hi < c1 ? sh.hi : c1;
-            if (lo >= hi) continue;
-            const T *w = static_cast<const T *>(p.down[__ldcg(p.chosen + c)]) + (size_t)n * p.expert_pitch;
-            acc += dot_row<T>(reinterpret_cast<const uint4 *>(w), smem, plane1, lo - c0, hi - c0, c0, lane);
-        }
-        acc = warp_sum(acc);
-        if (lane == 0) part[it] = acc;
-    }
+        return it;
+    });
     __syncthreads();
     for (int r = tid; r < rows; r += kThreads) {
         float a = 0.f;
-        for (int i = 0; i < ks; i++) a += part[(r << p.ksplit_log2) + i];
+        for (int i = 0; i < slots; i++) a += part[r * slots + i];
         const int n = r_lo + r;
         if (p.bias) a += to_f32(static_cast<const T *>(p.bias)[n]);
         p.x[n] = __ldcg(p.x + n) + a;
     }
 }
 
-// Grid and warps per row for `rows` weight rows of `pieces` 16-byte pieces: up to two CTAs per SM
-// (one when the inputs fill the shared memory), and the smallest split that spreads the rows
-// evenly over the warps without leaving a warp less than one full round of loads.
+// Grid and stretches per row for `units` of `rows_per_unit` weight rows of `pieces` 16-byte pieces:
+// up to two CTAs per SM (one when the inputs fill the shared memory), and the split that spreads the
+// rows most evenly over the warps at the least bookkeeping.
 struct Shape {
-    int grid, log2, rows_cap;
+    int grid, split, rows_cap;
 };
+int grid_for(const tlc_ctx *ctx, int units, long items, size_t input_bytes) {
+    int grid = (input_bytes > 96 * 1024 ? 1 : 2) * ctx->sm_count;
+    const long want = (items + kWarps - 1) / kWarps;
+    if (want < grid) grid = (int)want;
+    if (grid > units) grid = units;
+    return grid < 1 ? 1 : grid;
+}
 Shape choose_shape(const tlc_ctx *ctx, int units, int rows_per_unit, int pieces, size_t input_bytes) {
-    const int per_sm = input_bytes > 96 * 1024 ? 1 : 2;
-    Shape best{1, 0, 0};
+    Shape best{1, 1, 0};
     double best_cost = 1e30;
-    for (int log2 = 0; log2 <= 4; log2++) {
-        if (log2 > 0 && (pieces >> log2) < 32) break;
-        int grid = per_sm * ctx->sm_count;
-        const long items = (long)units * rows_per_unit << log2;
-        const long want = (items + kWarps - 1) / kWarps;
-        if (want < grid) grid = (int)want;
-        if (grid > units) grid = units;
-        if (grid < 1) grid = 1;
+    for (int split = 1; split <= 16; split *= 2) {
+        if (split > 1 && pieces / split < 32) break;
+        const int grid = grid_for(ctx, units, (long)units * rows_per_unit * split, input_bytes);
         const int cap = (units + grid - 1) / grid * rows_per_unit;
-        const int per_warp = ((cap << log2) + kWarps - 1) / kWarps;
-        // loads a lane makes one after the other, plus the cost of reducing and storing an item
-        const int rounds = (((pieces + (1 << log2) - 1) >> log2) + 32 * kUnroll - 1) / (32 * kUnroll);
-        const double loads = (double)((pieces + (1 << log2) - 1) >> log2) / 32.0;
-        const double cost = per_warp * (loads + 1.5 * rounds + 2.0);
+        const int per_warp = (cap * split + kWarps - 1) / kWarps;
+        const double batches = (double)(((pieces + split - 1) / split + 32 * kBatch - 1) / (32 * kBatch));
+        const double cost = per_warp * (batches + 0.5);  // an item's reduction costs about half a batch
         if (cost < best_cost * 0.98) {
             best_cost = cost;
-            best = {grid, log2, cap};
+            best = {grid, split, cap};
         }
     }
     return best;
 }
+// Stretches of a segment of `pieces` in the output kernel: two batches of a lane each.
+int split_for(int pieces) { return pieces <= 256 ? 1 : (pieces + 255) / 256; }
 
 template <typename K>
 int32_t set_limits(K kernel, bool (&done)[64], int device) {
@@ -385,8 +527,7 @@ int32_t set_limits(K kernel, bool (&done)[64], int device) {
 
 }  // namespace
 
-bool gemv_fits(int k) { return (size_t)2 * (k + 8) * sizeof(float) <= kSmemMax; }
-bool out_gemv_fits(int64_t k_total) { return (size_t)k_total * sizeof(float) <= kSmemMax; }
+bool gemv_fits(int k) { return (size_t)4 * (k + 8) * sizeof(float) <= kSmemMax; }
 
 #define TLC_LAUNCHED(ctx, le, what)                                                            \
     do {                                                                                       \
@@ -408,11 +549,11 @@ int32_t launch_gemv(tlc_ctx *ctx, GemvParams &p) {
     }
     p.v_total = v;
     const int pieces = (p.k + Vec<T>::N - 1) / Vec<T>::N;
-    const size_t input = (size_t)2 * pieces * 16 / sizeof(T) * sizeof(float);
+    const size_t input = (size_t)2 * pieces * 16 / sizeof(T) * sizeof(float) + (p.xn ? 0 : (size_t)2 * pieces * 16);
     const Shape sh = choose_shape(ctx, v / 2, 2, pieces, input);
-    p.ksplit_log2 = sh.log2;
+    p.split = sh.split;
     p.rows_cap = sh.rows_cap;
-    const size_t smem = input + ((size_t)sh.rows_cap << sh.log2) * sizeof(float);
+    const size_t smem = input + (size_t)sh.rows_cap * sh.split * sizeof(float);
     TLC_REQUIRE(smem <= kSmemMax + 16 * 1024, TLC_ERR_INVALID_OPERATION, "dense gemv: %d inputs do not fit the shared memory", p.k);
     p.prefetch = (int)(96 * 1024 / ((size_t)pieces * 16));
     cudaError_t le = tlc_launch_pdl(ctx, gemv_kernel<T>, dim3(sh.grid), dim3(kThreads), smem, p);
@@ -420,20 +561,57 @@ int32_t launch_gemv(tlc_ctx *ctx, GemvParams &p) {
     return TLC_OK;
 }
 
+// Shapes of the two launches below and the shared memory they take.
+template <typename T>
+static size_t plan_expert(const tlc_ctx *ctx, ExpertParams &p, int *grid) {
+    const int pieces = (p.k + Vec<T>::N - 1) / Vec<T>::N;
+    const size_t input = (size_t)pieces * 16 / sizeof(T) * sizeof(float);
+    const Shape sh = choose_shape(ctx, p.top * p.ff, 2, pieces, input);
+    p.split = sh.split;
+    p.rows_cap = sh.rows_cap;
+    *grid = sh.grid;
+    return input + (size_t)sh.rows_cap * sh.split * sizeof(float) + ((size_t)p.experts + 2 * p.top) * 4 + (size_t)2 * p.top * sizeof(void *) + 8;
+}
+template <typename T>
+static size_t plan_out(const tlc_ctx *ctx, OutParams &p, int *grid) {
+    int c = 0, slots = 0;
+    int64_t dense_bytes = 0;
+    for (int s = 0; s < p.n_seg; s++) {
+        const int pieces = (p.seg[s].k + Vec<T>::N - 1) / Vec<T>::N;
+        p.seg[s].c0 = c;
+        p.seg[s].split = split_for(pieces);
+        c += pieces;
+        slots += p.seg[s].split;
+        dense_bytes += (int64_t)pieces * 16;
+    }
+    p.expert_c0 = c;
+    p.expert_pieces = (p.expert_k + Vec<T>::N - 1) / Vec<T>::N;
+    p.expert_split = p.top ? split_for(p.expert_pieces) : 1;
+    p.pieces = c + p.top * p.expert_pieces;
+    slots += p.top * p.expert_split;
+    const size_t input = (size_t)p.pieces * Vec<T>::N * sizeof(float);
+    *grid = grid_for(ctx, p.n, (long)p.n * slots, input);
+    p.rows_cap = (p.n + *grid - 1) / *grid;
+    p.prefetch = dense_bytes ? (int)(128 * 1024 / dense_bytes) : 0;
+    return input + ((size_t)p.rows_cap * slots + 1) * sizeof(float) + (size_t)p.top * sizeof(void *) + 8;
+}
+
+template <typename T>
+bool layer_gemv_fits(const tlc_ctx *ctx, ExpertParams e, OutParams o) {
+    int grid;
+    if (e.top > 0 && (e.top > kThreads || plan_expert<T>(ctx, e, &grid) > kSmemMax + 16 * 1024)) return false;
+    return plan_out<T>(ctx, o, &grid) <= kSmemMax + 16 * 1024;
+}
+
 template <typename T>
 int32_t launch_expert_gemv(tlc_ctx *ctx, ExpertParams &p) {
     static bool done[64] = {};
     if (int32_t rc = set_limits(expert_gemv_kernel<T>, done, ctx->device)) return rc;
-    const int pieces = (p.k + Vec<T>::N - 1) / Vec<T>::N;
-    const size_t input = (size_t)pieces * 16 / sizeof(T) * sizeof(float);
-    const Shape sh = choose_shape(ctx, p.top * p.ff, 2, pieces, input);
-    p.ksplit_log2 = sh.log2;
-    p.rows_cap = sh.rows_cap;
-    const size_t smem = input + ((size_t)sh.rows_cap << sh.log2) * sizeof(float) + ((size_t)p.experts + 2 * p.top) * 4;
+    int grid = 1;
+    const size_t smem = plan_expert<T>(ctx, p, &grid);
     TLC_REQUIRE(smem <= kSmemMax + 16 * 1024 && p.top <= kThreads, TLC_ERR_INVALID_OPERATION,
                 "expert gemv: %d inputs do not fit the shared memory", p.k);
-    // Without dependent launch the kernels run one after the other anyway; the wait is then a no-op.
-    cudaError_t le = tlc_launch_pdl(ctx, expert_gemv_kernel<T>, dim3(sh.grid), dim3(kThreads), smem, p, 0);
+    cudaError_t le = tlc_launch_pdl(ctx, expert_gemv_kernel<T>, dim3(grid), dim3(kThreads), smem, p);
     TLC_LAUNCHED(ctx, le, "expert gemv");
     return TLC_OK;
 }
@@ -442,30 +620,17 @@ template <typename T>
 int32_t launch_out_gemv(tlc_ctx *ctx, OutParams &p) {
     static bool done[64] = {};
     if (int32_t rc = set_limits(out_gemv_kernel<T>, done, ctx->device)) return rc;
-    int c = 0;
-    int64_t dense_bytes = 0;
-    for (int s = 0; s < p.n_seg; s++) {
-        p.seg[s].c0 = c;
-        const int pieces = (p.seg[s].k + Vec<T>::N - 1) / Vec<T>::N;
-        c += pieces;
-        dense_bytes += (int64_t)pieces * 16;
-    }
-    p.expert_c0 = c;
-    p.expert_pieces = (p.expert_k + Vec<T>::N - 1) / Vec<T>::N;
-    p.pieces = c + p.top * p.expert_pieces;
-    const size_t input = (size_t)p.pieces * Vec<T>::N * sizeof(float);
-    const Shape sh = choose_shape(ctx, p.n, 1, p.pieces, input);
-    p.ksplit_log2 = sh.log2;
-    p.rows_cap = sh.rows_cap;
-    const size_t smem = input + ((size_t)sh.rows_cap << sh.log2) * sizeof(float);
-    TLC_REQUIRE(smem <= kSmemMax + 16 * 1024, TLC_ERR_INVALID_OPERATION, "output gemv: %d inputs do not fit the shared memory",
-                p.pieces * Vec<T>::N);
-    p.prefetch = dense_bytes ? (int)(128 * 1024 / dense_bytes) : 0;
-    cudaError_t le = tlc_launch_pdl(ctx, out_gemv_kernel<T>, dim3(sh.grid), dim3(kThreads), smem, p);
+    int grid = 1;
+    const size_t smem = plan_out<T>(ctx, p, &grid);
+    TLC_REQUIRE(smem <= kSmemMax + 16 * 1024 && p.top <= kThreads, TLC_ERR_INVALID_OPERATION,
+                "output gemv: %d inputs do not fit the shared memory", p.pieces * Vec<T>::N);
+    cudaError_t le = tlc_launch_pdl(ctx, out_gemv_kernel<T>, dim3(grid), dim3(kThreads), smem, p);
     TLC_LAUNCHED(ctx, le, "output gemv");
     return TLC_OK;
 }
 
+template bool layer_gemv_fits<bf16>(const tlc_ctx *, ExpertParams, OutParams);
+template bool layer_gemv_fits<float>(const tlc_ctx *, ExpertParams, OutParams);
 template int32_t launch_gemv<bf16>(tlc_ctx *, GemvParams &);
 template int32_t launch_gemv<float>(tlc_ctx *, GemvParams &);
 template int32_t launch_expert_gemv<bf16>(tlc_ctx *, ExpertParams &);

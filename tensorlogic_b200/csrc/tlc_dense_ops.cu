@@ -7,15 +7,51 @@ namespace tlc_dense {
 
 namespace {
 
+// Four neighbouring values.
+__device__ __forceinline__ void load4(const float *p, float (&f)[4]) {
+    const float4 v = *reinterpret_cast<const float4 *>(p);
+    f[0] = v.x;
+    f[1] = v.y;
+    f[2] = v.z;
+    f[3] = v.w;
+}
+__device__ __forceinline__ void load4(const bf16 *p, float (&f)[4]) {
+    const uint2 v = *reinterpret_cast<const uint2 *>(p);
+    f[0] = __uint_as_float(v.x << 16);
+    f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16);
+    f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+__device__ __forceinline__ void store4(float *p, const float (&f)[4]) {
+    *reinterpret_cast<float4 *>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+__device__ __forceinline__ void store4(bf16 *p, const float (&f)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+
 template <typename T>
 __global__ void embed_rows_kernel(const T *__restrict__ table, int64_t pitch, int vocab, int d, const int *__restrict__ ids,
                                   float *__restrict__ x) {
+    constexpr int N = Vec<T>::N;
     pdl_enter();  // ids are written by the previous step's sampling kernel
     const int r = blockIdx.y;
     int id = ids[r];
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; never read outside
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < d; i += gridDim.x * blockDim.x)
-        x[(size_t)r * d + i] = to_f32(table[(size_t)id * pitch + i]);
+    const T *src = table + (size_t)id * pitch;
+    float *dst = x + (size_t)r * d;
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * N;
+    if (i >= d) return;
+    float f[N];
+    unpack(__ldg(reinterpret_cast<const uint4 *>(src + i)), f);  // rows are padded to whole pieces
+    if ((d & 3) == 0 && i + N <= d) {
+#pragma unroll
+        for (int e = 0; e < N; e += 4) *reinterpret_cast<float4 *>(dst + i + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < N; e++)
+            if (i + e < d) dst[i + e] = f[e];
+    }
 }
 
 // One CTA per row.
@@ -29,6 +65,52 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const NormParams p) {
         for (int i = blockIdx.x * blockDim.x + tid; i < p.n_zero; i += gridDim.x * blockDim.x) p.zero[i] = 0;
     const int src = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
     float *x = p.x + (size_t)src * p.d;
+    if ((p.d & 3) == 0) {  // rows start on 16-byte boundaries
+        float s = 0.f;
+        for (int i = 4 * tid; i < p.d; i += 4 * blockDim.x) {
+            float4 v = __ldcg(reinterpret_cast<const float4 *>(x + i));
+            if (p.y) {
+                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int t = 0; t < p.top; t++) {
+                    float f[4];
+                    load4(static_cast<const T *>(p.y) + (size_t)p.place[(size_t)src * p.top + t] * p.y_pitch + i, f);
+                    a.x += f[0];
+                    a.y += f[1];
+                    a.z += f[2];
+                    a.w += f[3];
+                }
+                v.x += a.x;
+                v.y += a.y;
+                v.z += a.z;
+                v.w += a.w;
+                if (!p.rows) *reinterpret_cast<float4 *>(x + i) = v;
+            }
+            *reinterpret_cast<float4 *>(row + i) = v;
+            s += (v.x + v.y) + (v.z + v.w);
+        }
+        const float mean = block_sum(s, red) / (float)p.d;
+        float q = 0.f;
+        for (int i = 4 * tid; i < p.d; i += 4 * blockDim.x) {
+            const float4 v = *reinterpret_cast<const float4 *>(row + i);
+            const float a = v.x - mean, b = v.y - mean, c = v.z - mean, e = v.w - mean;
+            q += (a * a + b * b) + (c * c + e * e);
+        }
+        const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)p.d + p.eps);
+        for (int i = 4 * tid; i < p.d; i += 4 * blockDim.x) {
+            const float4 v = *reinterpret_cast<const float4 *>(row + i);
+            const float h[4] = {(v.x - mean) * rstd, (v.y - mean) * rstd, (v.z - mean) * rstd, (v.w - mean) * rstd};
+#pragma unroll
+            for (int o = 0; o < 2; o++) {
+                if (!p.w[o]) continue;
+                float f[4];
+                load4(static_cast<const T *>(p.w[o]) + i, f);
+#pragma unroll
+                for (int e = 0; e < 4; e++) f[e] *= h[e];
+                store4(static_cast<T *>(p.out[o]) + (size_t)blockIdx.x * p.ldo + i, f);
+            }
+        }
+        return;
+    }
     float s = 0.f;
     for (int i = tid; i < p.d; i += blockDim.x) {
         float v = __ldcg(x + i);
@@ -104,6 +186,71 @@ __global__ void __launch_bounds__(256) qk_rotate_kernel(const RotParams p) {
         const int head = i / p.Dp, e = i - head * p.Dp;
         kc[i] = from_f32<T>(e < p.D ? value(k, p.kn, rk, head, e) : 0.f);
         vc[i] = e < p.D ? k[head * p.D + e] : from_f32<T>(0.f);
+    }
+}
+
+// The same with 16-byte pieces, for bf16 heads of whole pieces whose rotated halves are whole pieces.
+// A unit is two pieces that turn against each other, or one piece behind the rotated part.
+__global__ void __launch_bounds__(256) qk_rotate_pieces_kernel(const RotParams p) {
+    extern __shared__ float cs[];  // [rot / 2] cos, [rot / 2] sin
+    __shared__ float red[33];
+    pdl_enter();
+    const int tid = threadIdx.x, r = blockIdx.x;
+    const bf16 *q = static_cast<const bf16 *>(p.q) + (size_t)r * p.ldq, *k = static_cast<const bf16 *>(p.k) + (size_t)r * p.ldk;
+    const int pos = p.pos[r], nq = p.H * p.D, nk = p.G * p.D, half = p.rot / 2;
+    float *sn = cs + half;
+    for (int i = tid; i < half; i += blockDim.x) sincosf((float)pos * p.freq[i], &sn[i], &cs[i]);
+    auto squares = [&](const bf16 *x, int n) {
+        float s = 0.f;
+        for (int i = tid; i < n / 8; i += blockDim.x) {
+            float f[8];
+            unpack(*(reinterpret_cast<const uint4 *>(x) + i), f);
+#pragma unroll
+            for (int e = 0; e < 8; e++) s += f[e] * f[e];
+        }
+        return s;
+    };
+    const float sq = squares(q, nq), sk = squares(k, nk);
+    const float rq = 1.0f / sqrtf(block_sum(sq, red) / (float)nq + p.eps);
+    const float rk = 1.0f / sqrtf(block_sum(sk, red) / (float)nk + p.eps);  // also a barrier behind cs / sn
+    const bool in_cache = pos >= 0 && pos < p.max_seq;
+    if (!in_cache && tid == 0 && atomicCAS(&p.status->code, 0, TLC_DEV_INDEX) == 0) p.status->where = 401;
+    const size_t base = ((size_t)p.slot[r] * p.max_seq + (in_cache ? pos : 0)) * p.G * p.D;
+    bf16 *kc = static_cast<bf16 *>(p.kc) + base, *vc = static_cast<bf16 *>(p.vc) + base;
+    bf16 *qo = static_cast<bf16 *>(p.q_out) + (size_t)r * nq;
+    const int turning = half / 8, units = turning + (p.D - p.rot) / 8;  // per head
+    const int all = (in_cache ? p.H + p.G : p.H) * units;
+    for (int u = tid; u < all; u += blockDim.x) {
+        const int head = u / units, i = u - head * units;
+        const bool is_q = head < p.H;
+        const int hb = (is_q ? head : head - p.H) * p.D, e = i < turning ? 8 * i : p.rot + 8 * (i - turning);
+        const bf16 *src = (is_q ? q : k) + hb, *w = static_cast<const bf16 *>(is_q ? p.qn : p.kn) + hb;
+        const float scale = is_q ? rq : rk;
+        bf16 *dst = (is_q ? qo : kc) + hb;
+        const uint4 raw0 = *reinterpret_cast<const uint4 *>(src + e);
+        float a[8], wa[8];
+        unpack(raw0, a);
+        unpack(__ldg(reinterpret_cast<const uint4 *>(w + e)), wa);
+#pragma unroll
+        for (int j = 0; j < 8; j++) a[j] = a[j] * scale * wa[j];
+        if (!is_q) *reinterpret_cast<uint4 *>(vc + hb + e) = raw0;
+        if (i < turning) {
+            const uint4 raw1 = *reinterpret_cast<const uint4 *>(src + e + half);
+            float b[8], wb[8];
+            unpack(raw1, b);
+            unpack(__ldg(reinterpret_cast<const uint4 *>(w + e + half)), wb);
+            if (!is_q) *reinterpret_cast<uint4 *>(vc + hb + e + half) = raw1;
+#pragma unroll
+            for (int j = 0; j < 8; j++) {
+                const float x = a[j], y = b[j] * scale * wb[j];
+                a[j] = x * cs[e + j] - y * sn[e + j];
+                b[j] = y * cs[e + j] + x * sn[e + j];
+            }
+            store4(dst + e + half, *reinterpret_cast<const float(*)[4]>(b));
+            store4(dst + e + half + 4, *reinterpret_cast<const float(*)[4]>(b + 4));
+        }
+        store4(dst + e, *reinterpret_cast<const float(*)[4]>(a));
+        store4(dst + e + 4, *reinterpret_cast<const float(*)[4]>(a + 4));
     }
 }
 
@@ -197,7 +344,7 @@ __global__ void __launch_bounds__(256) permute_kernel(const PermuteParams p) {
 
 template <typename T>
 int32_t launch_embed(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int m, float *x) {
-    const int d = (int)table->n_cols, per = (d + 1023) / 1024;
+    const int d = (int)table->n_cols, per = (d + 256 * Vec<T>::N - 1) / (256 * Vec<T>::N);
     cudaError_t le = tlc_launch_pdl(ctx, embed_rows_kernel<T>, dim3(per, m), dim3(256), 0, static_cast<const T *>(table->data),
                                     (int64_t)(table->row_pitch / sizeof(T)), (int)table->n_rows, d, ids, x);
     TLC_LAUNCHED(ctx, le, "embedding");
@@ -220,6 +367,11 @@ int32_t launch_norm(tlc_ctx *ctx, const NormParams &p) {
 
 template <typename T>
 int32_t launch_qk_rotate(tlc_ctx *ctx, const RotParams &p, int m) {
+    if (sizeof(T) == 2 && p.D % 8 == 0 && p.rot % 16 == 0) {
+        cudaError_t le = tlc_launch_pdl(ctx, qk_rotate_pieces_kernel, dim3(m), dim3(256), (size_t)p.rot * sizeof(float) + 16, p);
+        TLC_LAUNCHED(ctx, le, "query/key norm");
+        return TLC_OK;
+    }
     cudaError_t le = tlc_launch_pdl(ctx, qk_rotate_kernel<T>, dim3(m), dim3(256), (size_t)p.rot * sizeof(float) + 16, p);
     TLC_LAUNCHED(ctx, le, "query/key norm");
     return TLC_OK;

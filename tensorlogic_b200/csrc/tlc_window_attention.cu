@@ -245,19 +245,53 @@ __global__ void __launch_bounds__(kAttn) window_prefill_kernel(const __grid_cons
     }
 }
 
-// Merge area of one CTA: from every split the 16 rows' maximum and sum and this CTA's columns.
-__host__ __device__ constexpr int merge_floats(int D, int nsplit) { return nsplit * 16 * (D / nsplit + 2); }
+// Merge area of one CTA: from every split this CTA's columns of the 16 rows, each followed by the
+// row's maximum and sum (and two unused floats: rows are whole 16-byte pieces).
+__host__ __device__ constexpr int merge_floats(int D, int nsplit) { return nsplit * 16 * (D / nsplit + 4); }
 __host__ __device__ constexpr size_t decode_tile_bytes(int D) { return (size_t)4 * kKeys * (D + 8) * 2; }
 __host__ __device__ constexpr size_t decode_smem(int D, int nsplit, int half) {
     return decode_tile_bytes(D) + (size_t)16 * (D + 8) * 2 + (size_t)2 * (D + 8) * 2 + (size_t)2 * half * 4 +
-           (size_t)merge_floats(D, nsplit) * 4 + 64;
+           (size_t)merge_floats(D, nsplit) * 4 + 80;
 }
 
-__device__ __forceinline__ void store_remote(uint32_t addr, int rank, float v) {
+__device__ __forceinline__ uint32_t remote_address(uint32_t addr, int rank) {
     uint32_t dst;
     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(addr), "r"(rank));
-    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(v) : "memory");
+    return dst;
 }
+__device__ __forceinline__ void store_remote(uint32_t addr, float4 v) {
+    asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(v.x), "f"(v.y), "f"(v.z), "f"(v.w)
+                 : "memory");
+}
+__device__ __forceinline__ void store_remote(uint32_t addr, float2 v) {
+    asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(v.x), "f"(v.y) : "memory");
+}
+// Two sums over the block at once, the same values in every thread.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2 *red) {
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+    __syncthreads();
+    float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < kAttn / 32; i++) {
+        s.x += red[i].x;
+        s.y += red[i].y;
+    }
+    return s;
+}
+// Entries a pair unit covers: unit i < rot / 2 turns entries i and i + rot / 2, later units hold two
+// neighbours behind the rotated part.
+struct Pair {
+    int e0, e1;
+    bool turn;
+    __device__ __forceinline__ Pair(int i, int rot) {
+        const int half = rot / 2;
+        turn = i < half;
+        e0 = turn ? i : rot + 2 * (i - half);
+        e1 = turn ? i + half : e0 + 1;
+    }
+};
 
 template <int D>
 __global__ void __launch_bounds__(kAttn) window_decode_kernel(const __grid_constant__ WindowAttn p) {
@@ -269,8 +303,9 @@ __global__ void __launch_bounds__(kAttn) window_decode_kernel(const __grid_const
     bf16 *newk = qs + 16 * PITCH, *newv = newk + PITCH;
     const int half = p.rot / 2;
     float *cs = reinterpret_cast<float *>(newv + PITCH), *sn = cs + half;
-    float *merge = sn + half;           // [nsplit][16][D / nsplit + 2]
-    __shared__ float red[33], sm_m[4][16], sm_l[4][16];
+    float *merge = reinterpret_cast<float *>((reinterpret_cast<uintptr_t>(sn + half) + 15) & ~(uintptr_t)15);
+    __shared__ float2 red[kAttn / 32];
+    __shared__ float sm_m[4][16], sm_l[4][16];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int nsplit = p.nsplit;
     const bool cluster = nsplit > 1;
@@ -302,51 +337,81 @@ __global__ void __launch_bounds__(kAttn) window_decode_kernel(const __grid_const
         }
         cp_async_commit();
     };
-    // cache rows of earlier steps do not depend on the kernels in flight
+    // cache rows of earlier steps, norm weights and angles do not depend on the kernels in flight
     if (t_lo < t_hi) load_tile(t_lo, 0);
+    constexpr int NP = D / 16;  // pair units of the 16 query rows per thread; one of the key
+    const bool owner = newest / kKeys >= t_lo && newest / kKeys < t_hi;
+    const bf16 *qn = static_cast<const bf16 *>(p.qn) + (size_t)(hk * grp + 16 * qt) * p.D;
+    const bf16 *kn = static_cast<const bf16 *>(p.kn) + (size_t)hk * p.D;
+    bf16 qw[NP][2], kw[2];
+#pragma unroll
+    for (int j = 0; j < NP; j++) {
+        const int u = tid + kAttn * j, row = u / (D / 2);
+        const Pair pr(u % (D / 2), p.rot);
+        qw[j][0] = row < heads && pr.e0 < p.D ? qn[row * p.D + pr.e0] : from_f32<bf16>(0.f);
+        qw[j][1] = row < heads && pr.e1 < p.D ? qn[row * p.D + pr.e1] : from_f32<bf16>(0.f);
+    }
+    const Pair kp(tid, p.rot);
+    const bool kin = owner && tid < D / 2;
+    kw[0] = kin && kp.e0 < p.D ? kn[kp.e0] : from_f32<bf16>(0.f);
+    kw[1] = kin && kp.e1 < p.D ? kn[kp.e1] : from_f32<bf16>(0.f);
     for (int i = tid; i < half; i += kAttn) sincosf((float)pos * p.freq[i], &sn[i], &cs[i]);
     pdl_enter();
 
     const bf16 *q = static_cast<const bf16 *>(p.q) + (size_t)r * p.ldq, *kr = static_cast<const bf16 *>(p.k_raw) + (size_t)r * p.ldk;
-    float rq, rk;
-    {
-        // the padding of the raw rows is zero
-        auto squares = [&](const bf16 *x, int n) {
-            float s = 0.f;
-            for (int i = tid; i < (n + 7) / 8; i += kAttn) {
-                float f[8];
-                unpack(__ldcg(reinterpret_cast<const uint4 *>(x) + i), f);
+    const bf16 *qg = q + (size_t)(hk * grp + 16 * qt) * p.D, *kg = kr + (size_t)hk * p.D;
+    bf16 qv[NP][2], kv[2];
 #pragma unroll
-                for (int e = 0; e < 8; e++) s += f[e] * f[e];
-            }
-            return s;
-        };
-        const float sq = squares(q, p.H * p.D), sk = squares(kr, p.G * p.D);
-        rq = 1.0f / sqrtf(block_sum(sq, red) / (float)(p.H * p.D) + p.eps);
-        rk = 1.0f / sqrtf(block_sum(sk, red) / (float)(p.G * p.D) + p.eps);
+    for (int j = 0; j < NP; j++) {
+        const int u = tid + kAttn * j, row = u / (D / 2);
+        const Pair pr(u % (D / 2), p.rot);
+        qv[j][0] = row < heads && pr.e0 < p.D ? qg[row * p.D + pr.e0] : from_f32<bf16>(0.f);
+        qv[j][1] = row < heads && pr.e1 < p.D ? qg[row * p.D + pr.e1] : from_f32<bf16>(0.f);
     }
-    auto value = [&](const bf16 *src, const void *w, float scale, int head, int e) {
-        auto norm = [&](int at) { return to_f32(src[at]) * scale * to_f32(static_cast<const bf16 *>(w)[at]); };
-        const int at = head * p.D + e;
-        if (e >= p.rot) return norm(at);
-        const float v = norm(at);
-        return e < half ? v * cs[e] - norm(at + half) * sn[e] : v * cs[e - half] + norm(at - half) * sn[e - half];
+    kv[0] = kin && kp.e0 < p.D ? kg[kp.e0] : from_f32<bf16>(0.f);
+    kv[1] = kin && kp.e1 < p.D ? kg[kp.e1] : from_f32<bf16>(0.f);
+    auto squares = [&](const bf16 *x, int n) {  // rows are padded to whole pieces, with anything
+        float s = 0.f;
+        for (int i = tid; i < (n + 7) / 8; i += kAttn) {
+            float f[8];
+            unpack(__ldcg(reinterpret_cast<const uint4 *>(x) + i), f);
+#pragma unroll
+            for (int e = 0; e < 8; e++) s += 8 * i + e < n ? f[e] * f[e] : 0.f;
+        }
+        return s;
     };
-    for (int i = tid; i < 16 * D; i += kAttn) {
-        const int row = i / D, e = i % D;
-        qs[row * PITCH + e] = from_f32<bf16>(row < heads && e < p.D ? value(q, p.qn, rq, hk * grp + 16 * qt + row, e) : 0.f);
+    const float2 sq = block_sum2(squares(q, p.H * p.D), squares(kr, p.G * p.D), red);  // also the barrier behind cs / sn
+    const float rq = 1.0f / sqrtf(sq.x / (float)(p.H * p.D) + p.eps), rk = 1.0f / sqrtf(sq.y / (float)(p.G * p.D) + p.eps);
+    auto turn = [&](const Pair &pr, const bf16 (&v)[2], const bf16 (&w)[2], float scale, int i) {
+        const float a = to_f32(v[0]) * scale * to_f32(w[0]), b = to_f32(v[1]) * scale * to_f32(w[1]);
+        return pr.turn ? make_float2(a * cs[i] - b * sn[i], b * cs[i] + a * sn[i]) : make_float2(a, b);
+    };
+#pragma unroll
+    for (int j = 0; j < NP; j++) {
+        const int u = tid + kAttn * j, row = u / (D / 2), i = u % (D / 2);
+        const Pair pr(i, p.rot);
+        const float2 v = turn(pr, qv[j], qw[j], rq, i);
+        qs[row * PITCH + pr.e0] = from_f32<bf16>(v.x);
+        qs[row * PITCH + pr.e1] = from_f32<bf16>(v.y);
     }
-    const bool owner = newest >= 0 && newest / kKeys >= t_lo && newest / kKeys < t_hi;
-    if (owner)
-        for (int e = tid; e < D; e += kAttn) {
-            const bool in = e < p.D;
-            newk[e] = from_f32<bf16>(in ? value(kr, p.kn, rk, hk, e) : 0.f);
-            newv[e] = in ? kr[hk * p.D + e] : from_f32<bf16>(0.f);
-            if (qt == 0 && e < p.Dp) {
-                kbase[(size_t)pos * key_stride + e] = newk[e];
-                vbase[(size_t)pos * key_stride + e] = newv[e];
+    if (kin) {
+        const float2 v = turn(kp, kv, kw, rk, tid);
+        newk[kp.e0] = from_f32<bf16>(v.x);
+        newk[kp.e1] = from_f32<bf16>(v.y);
+        newv[kp.e0] = kv[0];
+        newv[kp.e1] = kv[1];
+        if (qt == 0) {
+            bf16 *kd = kbase + (size_t)pos * key_stride, *vd = vbase + (size_t)pos * key_stride;
+            if (kp.e0 < p.Dp) {
+                kd[kp.e0] = newk[kp.e0];
+                vd[kp.e0] = kv[0];
+            }
+            if (kp.e1 < p.Dp) {
+                kd[kp.e1] = newk[kp.e1];
+                vd[kp.e1] = kv[1];
             }
         }
+    }
     __syncthreads();
 
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
@@ -449,35 +514,33 @@ __global__ void __launch_bounds__(kAttn) window_decode_kernel(const __grid_const
         }
     }
     __syncthreads();
-    const int cols = D / nsplit, stride = cols + 2;
+    const int cols = D / nsplit, stride = cols + 4;
     const uint32_t merge_addr = (uint32_t)__cvta_generic_to_shared(merge);
     if (cluster) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");  // every peer is running
-    for (int i = tid; i < 16 * D; i += kAttn) {
-        const int row = i / D, e = i % D;
-        float m = fmaxf(fmaxf(sm_m[0][row], sm_m[1][row]), fmaxf(sm_m[2][row], sm_m[3][row]));
+    for (int i = tid; i < heads * (D / 4); i += kAttn) {
+        const int row = i / (D / 4), e = 4 * (i % (D / 4));
+        const float m = fmaxf(fmaxf(sm_m[0][row], sm_m[1][row]), fmaxf(sm_m[2][row], sm_m[3][row]));
         const float base = m == -INFINITY ? 0.f : m;
-        float a = 0.f, l = 0.f;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        float l = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; w++) {
             const float f = exp2f(sm_m[w][row] - base);
-            a += f * ow[(size_t)(w * 16 + row) * D + e];
+            const float4 v = *reinterpret_cast<const float4 *>(ow + (size_t)(w * 16 + row) * D + e);
+            a.x += f * v.x;
+            a.y += f * v.y;
+            a.z += f * v.z;
+            a.w += f * v.w;
             l += f * sm_l[w][row];
         }
-        const int dst = e / cols, c = e - dst * cols;
-        const uint32_t at = merge_addr + (uint32_t)(((split * 16 + row) * stride) * 4);
+        const int dst = e / cols, c = e - dst * cols, at = (split * 16 + row) * stride;
         if (cluster) {
-            store_remote(at + 4 * c, dst, a);
-            if (c == 0) {
-                store_remote(at + 4 * cols, dst, m);
-                store_remote(at + 4 * cols + 4, dst, l);
-            }
+            const uint32_t to = remote_address(merge_addr + 4 * at, dst);
+            store_remote(to + 4 * c, a);
+            if (c == 0) store_remote(to + 4 * cols, make_float2(m, l));
         } else {
-            float *mr = merge + (size_t)row * stride;
-            mr[c] = a;
-            if (c == 0) {
-                mr[cols] = m;
-                mr[cols + 1] = l;
-            }
+            *reinterpret_cast<float4 *>(merge + at + c) = a;
+            if (c == 0) *reinterpret_cast<float2 *>(merge + at + cols) = make_float2(m, l);
         }
     }
     if (cluster) {

@@ -121,6 +121,26 @@ def test_values_are_the_raw_keys(dev):
     check(dev, cfg, w, tokens(50, 61))
 
 
+@pytest.mark.parametrize("width,vocab", [(50, 61), (51, 130), (129, 33), (8, 9), (520, 40)])
+def test_widths(dev, width, vocab):
+    """Rows that are no whole number of 16-byte pieces; one and several wanted rows of a prompt."""
+    cfg = config([dense(attention(3, 1, 10, 12, 1, 6), 37), moe(attention(2, 2, 9, 5, 2, 4), 3, 1, 11, 5), attention(5, 1, 13, 9, 0, 12)],
+                 width=width, vocab=vocab)
+    w, seq = weights(cfg, width, gain=0.7), tokens(40, vocab)
+    check(dev, cfg, w, seq, dtypes=["float32"], tol=5.0)
+    want = ref.forward(cfg, w, seq)
+    for dtype in DTYPES:
+        dec = build(dev, cfg, w, dtype)
+        for place in (39, 17):
+            s = dec.open()
+            got = dec.feed(s, seq, [place])
+            dec.close(s)
+            assert error(got, want[[place]]) < (5 * TOL["float32"] if dtype == "float32" else 0.2)
+        tok, _ = dec.prefill(seq, return_logits=False)
+        row = want[-1]
+        assert row.max() - row[tok] < (1e-6 if dtype == "float32" else 0.2) * row.std()
+
+
 def test_norm_spans_the_whole_projection(dev):
     """One head's rows are twenty times the others': a norm per head would equalize them."""
     cfg = config([attention(4, 4, 16, window=30, keep=0)])
