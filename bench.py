@@ -28,6 +28,7 @@ says scaling "strong"; it is a different workload from the N=1 line.
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
 import os
 import subprocess
@@ -859,6 +860,8 @@ def run_toposun(args) -> None:
     from tensorlogic_b200.model import Llama, synthetic_model
     tokens, K, W = 2048, args.steps, max(args.warmup, 3)
     arch, twin = toposun_sizes()[args.size]
+    if args.window:
+        arch.layers = [dataclasses.replace(l, window=args.window) for l in arch.layers]
     if args.layers:
         arch.layers, twin.n_layers = arch.layers[:args.layers], min(args.layers, twin.n_layers)
     KP = max(3, min(K, 20))
@@ -923,7 +926,7 @@ def run_toposun(args) -> None:
         "steps": K, "warmup": W, "ms_per_step": ours["decode_ms"], "higher_is_better": True, "scaling": "weak",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
         "config": {"model": f"toposun-{args.size}", "layers": len(arch.layers), "width": arch.width, "global_batch": 1,
-                   "seq_len": tokens, "window": 1024, "parallelism": "single",
+                   "seq_len": tokens, "window": arch.layers[0].window, "parallelism": "single",
                    "l2": "the weights of a step exceed the 126 MB L2", "seed": SEED},
         "e2e": {"value": e2e, "unit": "tokens/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4},
         "gpu_launches": int(launches), "clocks": clock_line, "toposun": ours, "closest": closest,
@@ -940,6 +943,7 @@ def main() -> None:
                     help="micro-benchmark one kernel instead of the decode workload (see run_kernel)")
     ap.add_argument("--size", default="small", choices=["small", "wide", "experts"], help="of --workload toposun")
     ap.add_argument("--layers", type=int, default=0, help="--workload toposun: only the first so many layers (for profiles)")
+    ap.add_argument("--window", type=int, default=0, help="--workload toposun: another window than 1024")
     ap.add_argument("--no-closest", action="store_true", help="--workload toposun: leave the LLaMA runner out")
     ap.add_argument("--qtype", default="q4_0", choices=["q4_0", "q8_0"])
     ap.add_argument("--n", type=int, default=28672)

@@ -678,11 +678,11 @@ int32_t forward(tlc_decoder *D, const Pass &ps) {
     return D->cfg.dtype == TLC_TYPE_F32 ? forward_t<float>(D, ps) : forward_t<bf16>(D, ps);
 }
 
-int32_t sample(tlc_decoder *D, const float *logits, int rows, int fixed_pos, int *next, int *ids, int *positions, bool advance) {
+int32_t sample(tlc_decoder *D, const float *logits, int rows, int fixed_pos, int seq0, int *next, int *ids, int *positions, bool advance) {
     tlc_ctx *ctx = D->ctx;
     cudaError_t le = D->temperature > 0.0001f
                          ? tlc_launch_pdl(ctx, sample_advance_kernel<float>, dim3(rows), dim3(1024), 0, logits, D->cfg.vocab, 1,
-                                          rows, D->temperature, D->seed, (const float *)nullptr, fixed_pos, next, ids, positions,
+                                          rows, D->temperature, D->seed, (const float *)nullptr, fixed_pos, seq0, next, ids, positions,
                                           advance ? 1 : 0, D->report)
                          : tlc_launch_pdl(ctx, argmax_advance_kernel<float>, dim3(rows), dim3(1024), 0, logits, D->cfg.vocab, 1,
                                           rows, next, ids, positions, advance ? 1 : 0, D->report);
@@ -702,7 +702,7 @@ int32_t decode_step(tlc_decoder *D, int batch, bool advance) {
     ps.slot = D->slots;
     ps.decode = true;
     if (int32_t rc = forward(D, ps)) return rc;
-    return sample(D, D->logits, batch, -1, D->next_ids, D->ids, D->positions, advance);
+    return sample(D, D->logits, batch, -1, 0, D->next_ids, D->ids, D->positions, advance);
 }
 
 int32_t check_ids(const tlc_decoder *D, const int32_t *ids, int n) {
@@ -875,7 +875,7 @@ extern "C" int32_t tlc_decoder_prefill(tlc_decoder *D, int32_t seq, const int32_
             TLC_CUDA(cudaMemcpyAsync(logits_host + (size_t)done_want * D->cfg.vocab, D->logits, (size_t)w * D->cfg.vocab * 4,
                                      cudaMemcpyDeviceToHost, ctx->stream));
         if (draw) {
-            if (int32_t rc = sample(D, D->logits + (size_t)(rows - 1) * D->cfg.vocab, 1, pos0 + n - 1, D->next_ids + seq, nullptr,
+            if (int32_t rc = sample(D, D->logits + (size_t)(rows - 1) * D->cfg.vocab, 1, pos0 + n - 1, seq, D->next_ids + seq, nullptr,
                                     nullptr, false))
                 return rc;
             TLC_CUDA(cudaMemcpyAsync(D->ids + seq, D->next_ids + seq, 4, cudaMemcpyDeviceToDevice, ctx->stream));

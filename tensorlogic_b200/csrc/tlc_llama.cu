@@ -478,7 +478,7 @@ static int32_t forward(tlc_llama *L, int m, bool decode, int pos0, bool all_logi
                 L->temperature > 0.0001f
                     ? tlc_launch_pdl(ctx, sample_advance_kernel<__half>, dim3(srows), dim3(1024), 0, lg, L->vocab_local,
                                      c.tp_size, rows, L->temperature, L->sample_seed, (const float *)nullptr,
-                                     decode ? -1 : pos0 + m - 1, (int *)L->next_ids, (int *)L->ids, (int *)L->positions, advance ? 1 : 0,
+                                     decode ? -1 : pos0 + m - 1, 0, (int *)L->next_ids, (int *)L->ids, (int *)L->positions, advance ? 1 : 0,
                                      L->report)
                     : tlc_launch_pdl(ctx, argmax_advance_kernel<__half>, dim3(srows), dim3(1024), 0, lg, L->vocab_local,
                                      c.tp_size, rows, (int *)L->next_ids, (int *)L->ids, (int *)L->positions,
@@ -813,7 +813,7 @@ extern "C" int32_t tlc_temperature_sample(tlc_ctx *ctx, const void *logits_dev, 
         if (temperature > 0.0001f)
             sample_advance_kernel<__half><<<rows, 1024, 0, ctx->stream>>>(
                 static_cast<const __half *>(logits_dev), vocab, 1, rows, temperature, 0, (const float *)tlc_buf_ptr(ub),
-                -1, (int *)tlc_buf_ptr(ib), nullptr, nullptr, 0, HostReport{});
+                -1, 0, (int *)tlc_buf_ptr(ib), nullptr, nullptr, 0, HostReport{});
         else
             argmax_advance_kernel<__half><<<rows, 1024, 0, ctx->stream>>>(static_cast<const __half *>(logits_dev), vocab, 1, rows,
                                                                    (int *)tlc_buf_ptr(ib), nullptr, nullptr, 0, HostReport{});

@@ -132,11 +132,12 @@ __global__ void argmax_advance_kernel(const LT *__restrict__ logits, int vocab, 
 // run its starting sum, and the comparison is made against u * total instead of
 // dividing every probability (the f32 rounding differs from the sequential sum
 // only for draws within ~1e-6 of a boundary).
-// u comes from `uniforms[b]` when given, else from tlc_sample_uniform.
+// u comes from `uniforms[b]` when given, else from tlc_sample_uniform; row b belongs to sequence
+// seq0 + b.
 template <typename LT>
 __global__ void __launch_bounds__(1024) sample_advance_kernel(const LT *__restrict__ logits, int vocab, int shards,
                                                               int rows, float temperature, uint64_t seed,
-                                                              const float *__restrict__ uniforms, int fixed_pos,
+                                                              const float *__restrict__ uniforms, int fixed_pos, int seq0,
                                                               int *__restrict__ next_ids, int *__restrict__ ids,
                                                               int *__restrict__ positions, int advance, HostReport hr) {
     __shared__ float red[32];
@@ -184,7 +185,7 @@ __global__ void __launch_bounds__(1024) sample_advance_kernel(const LT *__restri
         wbase = __shfl_sync(0xffffffffu, wi - w, warp);  // exclusive sum of the warps before this one
     }
     const int pos = fixed_pos >= 0 ? fixed_pos : positions ? positions[b] : 0;  // position of the token fed to this step
-    const float u = uniforms ? uniforms[b] : tlc_sample_uniform(seed, (uint32_t)pos, (uint32_t)b);
+    const float u = uniforms ? uniforms[b] : tlc_sample_uniform(seed, (uint32_t)pos, (uint32_t)(seq0 + b));
     const float target = u * total;
     float run = wbase + incl - local;  // sum of everything before this thread's run
     if (target < run + local) {
