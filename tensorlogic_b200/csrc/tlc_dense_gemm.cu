@@ -4,7 +4,7 @@
 // bf16: persistent tcgen05 kernel.  A tile is 128 activation rows x 256 weight rows (a pair: 128
 // gate rows and the matching 128 up rows); both operands arrive by TMA in 64-wide K steps with the
 // 128-byte swizzle, four stages of 48 KB; one thread issues tcgen05.mma (M = 128, N = 256, K = 16)
-// into one of two 256-column accumulators in tensor memory, four warps drain the other one
+// into one of two 256-column accumulators in tensor memory, eight warps drain the other one
 // meanwhile.  Two stretches of K (attention output and feed-forward down) may add up in one
 // accumulator.  The tiles of a family of experts come from the row offsets the router left in
 // device memory.
@@ -22,7 +22,8 @@ namespace {
 
 constexpr int kStagesD = 4;
 constexpr int kABytes = 128 * 128, kBBytes = 256 * 128, kStageBytesD = kABytes + kBBytes;
-constexpr int kThreadsD = 192;  // TMA warp, MMA warp, four epilogue warps
+constexpr int kEpilogueWarps = 8;  // two per lane quarter of the tensor memory, taking the column pieces in turn
+constexpr int kThreadsD = 32 * (2 + kEpilogueWarps);  // and the TMA warp, the MMA warp
 constexpr size_t kSmemD = 1024 + (size_t)kStagesD * kStageBytesD + 256 + (size_t)(2 * kMaxSlots + 4) * sizeof(int);
 
 // Instruction descriptor: bf16 x bf16 -> f32, both operands K-major, M = 128, N = 256.
@@ -179,7 +180,7 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
         }
         for (int a = 0; a < 2; a++) {
             mbar_init(&acc_full[a], 1);
-            mbar_init(&acc_empty[a], 4);
+            mbar_init(&acc_empty[a], kEpilogueWarps);
         }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -255,7 +256,7 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
             __syncwarp();
         }
     } else {
-        const int wq = warp & 3;  // tensor-memory lanes this warp may read: 32 wq ..
+        const int wq = warp & 3, turn = (warp - 2) >> 2;  // tensor-memory lanes this warp may read: 32 wq ..
         int slot = 0, it = 0;
         for (int t = blockIdx.x; t < n_tiles; t += gridDim.x, it++) {
             const Tile tl = tile_at<128, 256>(p, start, first_row, t, slot);
@@ -267,7 +268,7 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
             const bool pair = g.epi >= EPI_CLAMPED_GLU;
             const int pieces = pair ? 4 : 8;
 #pragma unroll 1
-            for (int c = 0; c < pieces; c++) {
+            for (int c = turn; c < pieces; c += kEpilogueWarps / 4) {
                 if (tl.n0 + 32 * c >= g.n) break;
                 uint32_t r[32], u[32];
                 const uint32_t at = tmem + ((uint32_t)(32 * wq) << 16) + 256 * a + 32 * c;
