@@ -193,6 +193,15 @@ PROTOTYPES = {
 }
 
 _lib = None
+_path = LIB_PATH
+
+
+def use(path: str) -> None:
+    """Loads ``path`` (a part of the library, tensorlogic_b200.build.PARTS) instead of the whole library."""
+    global _path
+    if _lib is not None and path != _path:
+        raise RuntimeError(f"{_path} is loaded already")
+    _path = path
 
 
 def load() -> C.CDLL:
@@ -200,12 +209,14 @@ def load() -> C.CDLL:
     global _lib
     if _lib is not None:
         return _lib
-    if not os.path.exists(LIB_PATH):
+    if not os.path.exists(_path):
         raise ImportError(
-            f"{LIB_PATH} is missing: build it with `python -m tensorlogic_b200.build` "
+            f"{_path} is missing: build it with `python -m tensorlogic_b200.build` "
             "(needs nvcc); there is no fallback implementation")
-    lib = C.CDLL(LIB_PATH)
+    lib = C.CDLL(_path)
     for name, (res, args) in PROTOTYPES.items():
+        if _path != LIB_PATH and not hasattr(lib, name):
+            continue  # not in this part of the library
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args

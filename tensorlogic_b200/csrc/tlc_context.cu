@@ -213,6 +213,8 @@ extern "C" int32_t tlc_perf_report(tlc_ctx *ctx, char *buf, size_t buflen, int32
 extern "C" int32_t tlc_selftest_wait_timeout(tlc_ctx *ctx, int32_t kind) {
     if (int32_t rc = tlc_enter(ctx)) return rc;
     TLC_REQUIRE(kind >= 0 && kind <= 2, TLC_ERR_INVALID_OPERATION, "selftest_wait_timeout: kind %d (0, 1 or 2)", kind);
+    TLC_REQUIRE(tlc_selftest_mbarrier_wait && tlc_selftest_peer_wait, TLC_ERR_INVALID_OPERATION,
+                "selftest_wait_timeout: not in this part of the library");
     return kind == 0 ? tlc_selftest_mbarrier_wait(ctx) : tlc_selftest_peer_wait(ctx, kind == 2);
 }
 

@@ -52,7 +52,6 @@ struct Layer {
     int m_egate = -1, m_eup = -1, m_edown = -1;
     int a_attn = -1, a_act = -1, a_acte = -1;                        // activations of this layer's widths
     int ff_width() const { return c.ff_kind == TLC_FF_MOE ? c.shared_ff : c.ff_kind ? c.ff : 0; }
-    int top() const { return c.ff_kind == TLC_FF_MOE ? c.top : 0; }
 };
 
 inline int round8(int n) { return (n + 7) & ~7; }

@@ -170,8 +170,9 @@ static inline size_t tlc_block_bytes(int32_t type) {
 // A dense F16 copy of a quantized tensor (device-side dequantization).
 int32_t tlc_qtensor_to_f16(tlc_ctx *ctx, tlc_qtensor *qt, tlc_qtensor **out);
 // Failure-detection self-tests: launch a kernel whose bounded wait must run out.
-int32_t tlc_selftest_mbarrier_wait(tlc_ctx *ctx);
-int32_t tlc_selftest_peer_wait(tlc_ctx *ctx, bool flagged_words);
+// (Absent from a part of the library that does not hold the kernels they test.)
+__attribute__((weak)) int32_t tlc_selftest_mbarrier_wait(tlc_ctx *ctx);
+__attribute__((weak)) int32_t tlc_selftest_peer_wait(tlc_ctx *ctx, bool flagged_words);
 // Makes the context's device current; every entry point calls it first.
 int32_t tlc_enter(tlc_ctx *ctx);
 // After a stream synchronize that followed a copy of the status word to host_status.

@@ -23,6 +23,7 @@ from .model import Llama, LlamaArch, load_model
 class Entry:
     dtypes: tuple[str, ...]              # what a runner can compute in; the first is the default
     load: Callable[..., object]          # (dev, path, config or None, dtype, options) -> runner
+    part: str | None = None              # the part of the library that is enough (build.PARTS); None: all of it
 
 
 def _llama(dev: Device, path: str, _config, _dtype: str, options: dict) -> Llama:
@@ -41,7 +42,7 @@ def _decoder(read_config) -> Callable[..., object]:
 
 ARCHITECTURES: dict[str, Entry] = {
     "llama": Entry(("float16",), _llama),
-    toposun.NAME: Entry(decoder.Decoder.dtypes, _decoder(toposun.read_config)),
+    toposun.NAME: Entry(decoder.Decoder.dtypes, _decoder(toposun.read_config), "decoder"),
 }
 
 

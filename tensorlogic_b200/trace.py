@@ -59,12 +59,13 @@ def replay(runner, lines, out_dir: str, say=print) -> None:
 
 def main(argv=None) -> int:
     args = _arguments(argv)
-    from . import registry
+    from . import _lib, build, registry
     from .api import Device
     name, _ = registry.identify(args.model)
     if args.dtype not in registry.ARCHITECTURES[name].dtypes:
         print(f"{name} models do not run in {args.dtype}", file=sys.stderr)
         return REFUSED
+    _lib.use(build.ensure(registry.ARCHITECTURES[name].part))  # compiles in a fresh checkout
     runner = registry.load(Device(args.device), args.model, args.dtype, max_seq=args.max_tokens, max_batch=args.max_requests,
                            max_prefill=min(args.max_tokens, 2048))
     replay(runner, sys.stdin, args.out, lambda s: print(s, flush=True))

@@ -66,6 +66,21 @@ def test_gguf_files_keep_their_class(tmp_path, lib):
     assert registry.identify(str(p)) == ("llama", None)
 
 
+def test_the_decoder_part_of_the_library_is_complete(lib):
+    """The part that serves decoder models alone loads and exports what their runner calls."""
+    import ctypes
+    import os
+    from tensorlogic_b200 import build, registry
+    assert registry.ARCHITECTURES["Toposun"].part == "decoder"
+    path = build.build(part="decoder")
+    assert path != build.LIB and os.path.exists(path)
+    part = ctypes.CDLL(path, mode=os.RTLD_NOW)
+    for name in ("tlc_init", "tlc_model_load_safetensors", "tlc_decoder_create", "tlc_decoder_prefill", "tlc_decoder_decode_host",
+                 "tlc_decoder_release", "tlc_synchronize"):
+        assert hasattr(part, name)
+    assert not hasattr(part, "tlc_llama_create")
+
+
 class FakeRunner:
     def __init__(self):
         self.free, self.seen, self.closed = [0], {}, []
