@@ -373,6 +373,10 @@ TLC_API int32_t tlc_kvcache_create(tlc_ctx *ctx, int32_t n_layers, int32_t max_b
 TLC_API int32_t tlc_kvcache_create_layers(tlc_ctx *ctx, int32_t type, int32_t n_layers, int32_t max_batch,
                                           int32_t max_seq, const int32_t *kv_heads, const int32_t *head_dims,
                                           tlc_kvcache **out);
+/* A cache of latents: layer l holds ONE row of row_values[l] values (a multiple of 8) per position, key and
+ * value of all heads in one; tlc_kvcache_layer_ptrs gives it as K, V is NULL. */
+TLC_API int32_t tlc_kvcache_create_latent(tlc_ctx *ctx, int32_t type, int32_t n_layers, int32_t max_batch,
+                                          int32_t max_seq, const int32_t *row_values, tlc_kvcache **out);
 TLC_API int32_t tlc_kvcache_destroy(tlc_kvcache *cache);
 TLC_API int32_t tlc_kvcache_layer_ptrs(tlc_kvcache *cache, int32_t layer, void **k_dev,
                                        void **v_dev);
@@ -569,21 +573,37 @@ TLC_API int32_t tlc_llama_decode_enqueue_parts(tlc_llama *l, int32_t batch, int3
 /* ---- config-driven decoder ---------------------------------------------------- */
 
 /* A decoder-only transformer whose layers are described one by one: the mechanisms below, with
- * their constants as parameters.  A layer adds its mixer, fed with one layer norm of the residual
- * x, and its feed-forward, fed with another layer norm of the same x, to x; x is kept in 32 bits,
- * weights and activations are BF16 or F32.
- * Mixer: grouped-query attention.  Biases on q, k and the output; the projected keys double as the
- * values; one RMS norm spans all query heads, one all key heads; then the first rot_dims entries
- * of a head turn, entry e with entry e + rot_dims/2, by position * rot_base^(-2e/rot_dims).  Key j
- * is visible to query i for 0 <= i - j < window, and for j <= i also when j < keep_first.
+ * their constants as parameters.  The residual is kept in 32 bits, weights and activations are
+ * BF16 or F32.  Two forms of a layer:
+ *   streams == 0  one residual x; a layer adds its mixer, fed with one layer norm of x, and its
+ *                 feed-forward, fed with another layer norm of the same x (window mixer);
+ *   streams > 0   so many residual streams x_s, all the embedding at first.  Mixer, then feed-forward
+ *                 (sublayers 1 and 2), each: u = sum_s in[s] x_s; y = scale * sublayer(norm(u));
+ *                 x_t <- sum_s mix[s][t] x_s + out[t] y.  norm(u) = tanh(alpha u) * w + b.  At the end
+ *                 x is the sum of the streams (latent mixer).
+ * The layers run in the order `runs` (layer numbers; a layer may run several times, every run has its
+ * own cache), or each once.
+ * Mixer (mixer):
+ *   TLC_MIX_WINDOW  grouped-query attention.  Biases on q, k and the output; the projected keys double
+ *                   as the values; one RMS norm spans all query heads, one all key heads; then the
+ *                   first rot_dims entries of a head turn, entry e with entry e + rot_dims/2, by
+ *                   position * rot_base^(-2e/rot_dims).  Key j is visible to query i for
+ *                   0 <= i - j < window, and for j <= i also when j < keep_first.
+ *   TLC_MIX_LATENT  queries through an RMS-normed latent of q_rank values, dim unrotated and rot_dims
+ *                   rotated entries per head (neighbours 2e, 2e + 1 turn); keys and values of all heads
+ *                   from one RMS-normed latent of kv_rank values per token, dim and vdim per head, and
+ *                   one rotated key part all heads share; causal; the softmax has one more term per
+ *                   head, exp(sink), in its denominator.
  * Feed-forward (ff_kind):
  *   TLC_FF_NONE          none;
  *   TLC_FF_CLAMPED_GLU   down(g sigmoid(1.702 g) (u + 1)), g = min(gate, limit), u = up cut to +-limit;
  *   TLC_FF_MOE           the `top` experts (silu(gate) * up) with the largest sigmoid scores, each fed
  *                        with its score times the input; shared_ff > 0: one more expert for every
- *                        token, times a sigmoid gate of its own.
- * Logits: the embedding table against the final layer norm. */
-enum { TLC_FF_NONE = 0, TLC_FF_CLAMPED_GLU = 1, TLC_FF_MOE = 2 };
+ *                        token, times a sigmoid gate of its own;
+ *   TLC_FF_SILU_GLU      down(silu(gate) * up), biases on all three (streams > 0).
+ * Logits: the embedding table against the final norm; logit_softcap c > 0: c * tanh(logit / c). */
+enum { TLC_FF_NONE = 0, TLC_FF_CLAMPED_GLU = 1, TLC_FF_MOE = 2, TLC_FF_SILU_GLU = 3 };
+enum { TLC_MIX_WINDOW = 0, TLC_MIX_LATENT = 1 };
 typedef struct tlc_decoder_layer {
     int32_t heads, kv_heads, dim;       /* query heads, key/value heads, size of a head     */
     int32_t window, keep_first;         /* sliding window and the first tokens it keeps     */
@@ -593,6 +613,8 @@ typedef struct tlc_decoder_layer {
     int32_t ff_kind, ff;                /* TLC_FF_*; ff: width of the dense feed-forward    */
     float limit;
     int32_t experts, top, expert_ff, shared_ff;
+    int32_t mixer;                      /* TLC_MIX_*                                        */
+    int32_t vdim, q_rank, kv_rank;      /* latent mixer                                     */
 } tlc_decoder_layer;
 typedef struct tlc_decoder_config {
     int32_t n_layers, width, vocab;
@@ -603,12 +625,19 @@ typedef struct tlc_decoder_config {
     int32_t max_prefill;     /* rows one pass takes; longer portions run in several        */
     int32_t max_logit_rows;  /* rows of logits one pass may be asked for                   */
     int32_t no_graph;
+    int32_t streams;         /* residual streams (at most 8), or 0                         */
+    float logit_softcap;     /* or 0                                                       */
+    int32_t n_runs;          /* entries of runs, or 0: every layer once                    */
     const tlc_decoder_layer *layers;
+    const int32_t *runs;
 } tlc_decoder_config;
 typedef struct tlc_decoder tlc_decoder;
 /* Binds a model's tensors by name: "embed", "final.norm" and per layer "l<i>." + norm1, norm2,
  * mix.{q,q.b,q.norm,k,k.b,k.norm,o,o.b}, mlp.{gate,up,down} or mlp.{router,e<j>.gate,e<j>.up,
- * e<j>.down,shared.gate,shared.up,shared.down,shared.sg}. The model must outlive the decoder. */
+ * e<j>.down,shared.gate,shared.up,shared.down,shared.sg}; with streams "embed", "final.norm" and per
+ * layer norm1, norm2, mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,sink,o}, mlp.{gate,up,down}[.b], ls1, ls2
+ * (the scales), hc1.{in,out,mix}, hc2.{in,out,mix}, every norm with .alpha and .b.  The model must
+ * outlive the decoder. */
 TLC_API int32_t tlc_decoder_create(tlc_ctx *ctx, tlc_model *model, const tlc_decoder_config *cfg, tlc_decoder **out);
 TLC_API int32_t tlc_decoder_destroy(tlc_decoder *d);
 /* The next n tokens of sequence `seq`, at positions pos0 .. pos0 + n - 1; pos0 must be where the

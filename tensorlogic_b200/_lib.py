@@ -18,7 +18,8 @@ ERR_ALLOCATION, ERR_LOAD, ERR_BUFFER_EXHAUSTED, ERR_INDEX = -5, -6, -7, -8
 ERR_INVALID_DIMENSION, ERR_TIMEOUT, ERR_COMM = -9, -10, -11
 
 TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0, TYPE_BF16 = 0, 1, 2, 8, 30
-FF_NONE, FF_CLAMPED_GLU, FF_MOE = 0, 1, 2
+FF_NONE, FF_CLAMPED_GLU, FF_MOE, FF_SILU_GLU = 0, 1, 2, 3
+MIX_WINDOW, MIX_LATENT = 0, 1
 SPLIT_NONE, SPLIT_ROWS, SPLIT_COLS = 0, 1, 2
 
 _ERROR_NAMES = {
@@ -56,14 +57,16 @@ class DecoderLayer(C.Structure):
     _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("window", C.c_int32),
                 ("keep_first", C.c_int32), ("rot_dims", C.c_int32), ("rot_base", C.c_double), ("scale", C.c_float),
                 ("ff_kind", C.c_int32), ("ff", C.c_int32), ("limit", C.c_float), ("experts", C.c_int32),
-                ("top", C.c_int32), ("expert_ff", C.c_int32), ("shared_ff", C.c_int32)]
+                ("top", C.c_int32), ("expert_ff", C.c_int32), ("shared_ff", C.c_int32), ("mixer", C.c_int32),
+                ("vdim", C.c_int32), ("q_rank", C.c_int32), ("kv_rank", C.c_int32)]
 
 
 class DecoderConfig(C.Structure):
     """tlc_decoder_config of include/tlcuda.h."""
     _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("norm_eps", C.c_float),
                 ("dtype", C.c_int32), ("max_seq", C.c_int32), ("max_batch", C.c_int32), ("max_prefill", C.c_int32),
-                ("max_logit_rows", C.c_int32), ("no_graph", C.c_int32), ("layers", C.POINTER(DecoderLayer))]
+                ("max_logit_rows", C.c_int32), ("no_graph", C.c_int32), ("streams", C.c_int32), ("logit_softcap", C.c_float),
+                ("n_runs", C.c_int32), ("layers", C.POINTER(DecoderLayer)), ("runs", C.POINTER(C.c_int32))]
 
 
 vp, i32, i64, u32, u64, sz, f32 = C.c_void_p, C.c_int32, C.c_int64, C.c_uint32, C.c_uint64, C.c_size_t, C.c_float
@@ -124,6 +127,7 @@ PROTOTYPES = {
     "tlc_linear_residual": (i32, [vp, vp, vp, i32, vp, vp]),
     "tlc_kvcache_create": (i32, [vp, i32, i32, i32, i32, i32, P(vp)]),
     "tlc_kvcache_create_layers": (i32, [vp, i32, i32, i32, i32, P(i32), P(i32), P(vp)]),
+    "tlc_kvcache_create_latent": (i32, [vp, i32, i32, i32, i32, P(i32), P(vp)]),
     "tlc_kvcache_destroy": (i32, [vp]),
     "tlc_kvcache_layer_ptrs": (i32, [vp, i32, P(vp), P(vp)]),
     "tlc_kvcache_append": (i32, [vp, vp, i32, vp, vp, i32, i32, vp]),

@@ -24,7 +24,8 @@ LIB = os.path.join(PKG, "libtlcuda.so")
 
 PARTS = {
     "decoder": ("tlc_context", "tlc_qtensor", "tlc_attention", "tlc_gguf", "tlc_safetensors", "tlc_decoder", "tlc_dense_gemv",
-                "tlc_dense_gemm", "tlc_dense_ops", "tlc_window_attention"),
+                "tlc_dense_gemm", "tlc_dense_ops", "tlc_window_attention", "tlc_latent_attention", "tlc_latent_prefill",
+                "tlc_decoder_streams"),
 }
 
 NVCC_FLAGS = [

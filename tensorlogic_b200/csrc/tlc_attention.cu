@@ -866,12 +866,12 @@ int32_t tlc_launch_attention(tlc_ctx *ctx, tlc_kvcache *cache, int layer, const 
     return TLC_OK;
 }
 
-// The two zero-filled arrays of a cache; frees `c` when they cannot be had.
-static int32_t kvcache_allocate(tlc_kvcache *c, size_t bytes) {
+// The two zero-filled arrays of a cache (latents: the first alone); frees `c` when they cannot be had.
+static int32_t kvcache_allocate(tlc_kvcache *c, size_t bytes, bool values = true) {
     cudaError_t e = cudaMalloc(&c->k, bytes);
-    if (e == cudaSuccess) e = cudaMalloc(&c->v, bytes);
+    if (e == cudaSuccess && values) e = cudaMalloc(&c->v, bytes);
     if (e == cudaSuccess) e = cudaMemsetAsync(c->k, 0, bytes, c->ctx->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(c->v, 0, bytes, c->ctx->stream);
+    if (e == cudaSuccess && values) e = cudaMemsetAsync(c->v, 0, bytes, c->ctx->stream);
     if (e != cudaSuccess) {
         cudaGetLastError();
         if (c->k) cudaFree(c->k);
@@ -935,6 +935,33 @@ extern "C" int32_t tlc_kvcache_create_layers(tlc_ctx *ctx, int32_t type, int32_t
     return TLC_OK;
 }
 
+extern "C" int32_t tlc_kvcache_create_latent(tlc_ctx *ctx, int32_t type, int32_t n_layers, int32_t max_batch,
+                                             int32_t max_seq, const int32_t *row_values, tlc_kvcache **out) {
+    if (int32_t rc = tlc_enter(ctx)) return rc;
+    TLC_REQUIRE(out && row_values, TLC_ERR_INVALID_OPERATION, "kvcache_create_latent: null pointer");
+    *out = nullptr;
+    TLC_REQUIRE(type == TLC_TYPE_BF16 || type == TLC_TYPE_F32, TLC_ERR_INVALID_OPERATION,
+                "kvcache_create_latent: type %d (bf16 or f32)", type);
+    TLC_REQUIRE(n_layers > 0 && max_batch > 0 && max_seq > 0, TLC_ERR_INVALID_DIMENSION, "kvcache_create_latent: bad shape");
+    for (int l = 0; l < n_layers; l++)
+        TLC_REQUIRE(row_values[l] > 0 && row_values[l] % 8 == 0, TLC_ERR_INVALID_DIMENSION, "kvcache_create_latent: bad layer %d", l);
+    tlc_kvcache *c = new tlc_kvcache();
+    c->ctx = ctx;
+    c->type = type;
+    c->elem = type == TLC_TYPE_F32 ? 4 : 2;
+    c->n_layers = n_layers;
+    c->max_batch = max_batch;
+    c->max_seq = max_seq;
+    size_t total = 0;
+    for (int l = 0; l < n_layers; l++) {
+        c->layers.push_back({1, row_values[l], row_values[l], total});
+        total += (size_t)max_batch * max_seq * row_values[l];
+    }
+    if (int32_t rc = kvcache_allocate(c, total * c->elem, false)) return rc;
+    *out = c;
+    return TLC_OK;
+}
+
 extern "C" int32_t tlc_kvcache_destroy(tlc_kvcache *cache) {
     if (!cache) return TLC_OK;
     cudaSetDevice(cache->ctx->device);
@@ -948,7 +975,7 @@ extern "C" int32_t tlc_kvcache_layer_ptrs(tlc_kvcache *cache, int32_t layer, voi
     TLC_REQUIRE(cache && layer >= 0 && layer < cache->n_layers, TLC_ERR_INDEX, "kvcache: bad layer %d", layer);
     const size_t off = cache->layers[(size_t)layer].offset * cache->elem;
     if (k_dev) *k_dev = reinterpret_cast<uint8_t *>(cache->k) + off;
-    if (v_dev) *v_dev = reinterpret_cast<uint8_t *>(cache->v) + off;
+    if (v_dev) *v_dev = cache->v ? reinterpret_cast<uint8_t *>(cache->v) + off : nullptr;
     return TLC_OK;
 }
 

@@ -22,8 +22,7 @@
 #include <cstring>
 #include <memory>
 
-#include "tlc_dense.cuh"
-#include "tlc_sample.cuh"
+#include "tlc_decoder.h"
 
 using namespace tlc_dense;
 using namespace tlc_sample;
@@ -31,66 +30,11 @@ using namespace tlc_sample;
 extern "C" int32_t tlc_model_get(tlc_model *, const char *, tlc_qtensor **);
 extern "C" int32_t tlc_kvcache_create_layers(tlc_ctx *, int32_t, int32_t, int32_t, int32_t, const int32_t *, const int32_t *,
                                              tlc_kvcache **);
+extern "C" int32_t tlc_kvcache_create_latent(tlc_ctx *, int32_t, int32_t, int32_t, int32_t, const int32_t *, tlc_kvcache **);
 extern "C" int32_t tlc_kvcache_destroy(tlc_kvcache *);
 extern "C" int32_t tlc_kvcache_layer_ptrs(tlc_kvcache *, int32_t, void **, void **);
 
-namespace {
-
-constexpr int kMaxSeqs = 64;
-
-struct Layer {
-    tlc_decoder_layer c;
-    tlc_qtensor *norm1 = nullptr, *norm2 = nullptr;
-    tlc_qtensor *q, *qb, *qn, *k, *kb, *kn, *o, *ob;
-    tlc_qtensor *gate = nullptr, *up = nullptr, *down = nullptr;  // dense or shared expert
-    tlc_qtensor *router = nullptr, *sg = nullptr;
-    std::vector<tlc_qtensor *> e_gate, e_up, e_down;
-    float *freq = nullptr;                                           // [rot_dims / 2]
-    const void **gate_tab = nullptr, **up_tab = nullptr, **down_tab = nullptr;  // device, per expert
-    // tensor maps by index (bf16)
-    int m_q = -1, m_k = -1, m_o = -1, m_gate = -1, m_up = -1, m_down = -1, m_router = -1, m_sg = -1;
-    int m_egate = -1, m_eup = -1, m_edown = -1;
-    int a_attn = -1, a_act = -1, a_acte = -1;                        // activations of this layer's widths
-    int ff_width() const { return c.ff_kind == TLC_FF_MOE ? c.shared_ff : c.ff_kind ? c.ff : 0; }
-};
-
-inline int round8(int n) { return (n + 7) & ~7; }
-
-}  // namespace
-
-struct tlc_decoder {
-    tlc_ctx *ctx;
-    tlc_decoder_config cfg;
-    std::vector<Layer> layers;
-    tlc_qtensor *embed, *final_norm;
-    tlc_kvcache *cache = nullptr;
-    size_t elem;
-    int rows, logit_rows, top_max = 0;
-    bool one_row_ok = true;     // every layer's inputs fit the one-row kernels
-    std::vector<void *> owned;  // device allocations
-    CUtensorMap *maps = nullptr;
-    int a_h1 = -1, a_h2 = -1, a_hp = -1, a_hf = -1, m_embed = -1;
-    // activations
-    float *x, *h_row, *router_out, *weight, *scale, *logits;
-    uint8_t *h1, *h2, *q_raw, *k_raw, *q_rot, *attn, *act, *hp, *act_e, *y, *hf;
-    int ldw, ld_router = 1;
-    int *chosen, *rank, *place, *count, *off;
-    // row metadata: of a prompt portion, and of the sequences (decode)
-    int *row_ids, *row_pos, *row_slot, *want;
-    int *ids, *positions, *next_ids, *slots;
-    int *host_rows = nullptr;     // pinned: ids, positions, slots, wanted rows
-    int *host_next = nullptr;     // pinned
-    int *host_ids = nullptr;      // pinned
-    const int *ids_src = nullptr; // set while the host step is captured
-    HostReport report{};
-    std::map<int, cudaGraphExec_t> graph;  // batch; 1000 + batch: the host step
-    int launches = 0;
-    std::vector<int> pos_hi;      // host-side upper bound of every sequence's position
-    float temperature = 0.f;
-    uint64_t seed = 0;
-};
-
-namespace {
+namespace tlc_dense {
 
 int32_t dev_alloc(tlc_decoder *D, void **p, size_t bytes) {
     cudaError_t e = cudaMalloc(p, bytes ? bytes : 16);
@@ -100,23 +44,27 @@ int32_t dev_alloc(tlc_decoder *D, void **p, size_t bytes) {
         return tlc_fail(TLC_ERR_ALLOCATION, "activation buffer of %zu bytes failed: %s", bytes, cudaGetErrorString(e));
     }
     D->owned.push_back(*p);
-    // padding columns are read as zeros; nothing is ever uninitialized
     TLC_CUDA(cudaMemsetAsync(*p, 0, bytes ? bytes : 16, D->ctx->stream));
     return TLC_OK;
 }
 
-template <typename P>
-int32_t upload(tlc_decoder *D, P **dst, const void *src, size_t bytes) {
-    void *p = nullptr;
-    if (int32_t rc = dev_alloc(D, &p, bytes)) return rc;
-    TLC_CUDA(cudaMemcpyAsync(p, src, bytes, cudaMemcpyHostToDevice, D->ctx->stream));
-    TLC_CUDA(cudaStreamSynchronize(D->ctx->stream));  // `src` may go away
-    *dst = static_cast<P *>(p);
+int32_t bind_tensor(tlc_decoder *D, tlc_model *model, const std::string &name, int64_t rows, int64_t cols, tlc_qtensor **t) {
+    if (int32_t rc = tlc_model_get(model, name.c_str(), t)) return rc;
+    TLC_REQUIRE((*t)->n_rows == rows && (*t)->n_cols == cols, TLC_ERR_SHAPE_MISMATCH,
+                "tensor '%s' is [%lld, %lld], expected [%lld, %lld]", name.c_str(), (long long)(*t)->n_rows,
+                (long long)(*t)->n_cols, (long long)rows, (long long)cols);
+    TLC_REQUIRE((*t)->type == D->cfg.dtype, TLC_ERR_LOAD, "tensor '%s' has type %d, the decoder runs in type %d", name.c_str(),
+                (*t)->type, D->cfg.dtype);
     return TLC_OK;
 }
 
+}  // namespace tlc_dense
+
+namespace {
+
 // Checks the configuration of one layer.
 int32_t check_layer(const tlc_decoder_layer &c, int i) {
+    TLC_REQUIRE(c.mixer == TLC_MIX_WINDOW, TLC_ERR_INVALID_OPERATION, "layer %d: mixer %d needs residual streams", i, c.mixer);
     TLC_REQUIRE(c.heads > 0 && c.kv_heads > 0 && c.dim > 0 && c.heads % c.kv_heads == 0, TLC_ERR_INVALID_DIMENSION,
                 "layer %d: %d heads over %d key/value heads of %d", i, c.heads, c.kv_heads, c.dim);
     TLC_REQUIRE(c.dim <= 512, TLC_ERR_INVALID_DIMENSION, "layer %d: heads of %d values (at most 512)", i, c.dim);
@@ -137,15 +85,7 @@ int32_t check_layer(const tlc_decoder_layer &c, int i) {
 
 int32_t bind(tlc_decoder *D, tlc_model *model) {
     const tlc_decoder_config &cfg = D->cfg;
-    auto get = [&](const std::string &name, int64_t rows, int64_t cols, tlc_qtensor **t) -> int32_t {
-        if (int32_t rc = tlc_model_get(model, name.c_str(), t)) return rc;
-        TLC_REQUIRE((*t)->n_rows == rows && (*t)->n_cols == cols, TLC_ERR_SHAPE_MISMATCH,
-                    "tensor '%s' is [%lld, %lld], expected [%lld, %lld]", name.c_str(), (long long)(*t)->n_rows,
-                    (long long)(*t)->n_cols, (long long)rows, (long long)cols);
-        TLC_REQUIRE((*t)->type == cfg.dtype, TLC_ERR_LOAD, "tensor '%s' has type %d, the decoder runs in type %d", name.c_str(),
-                    (*t)->type, cfg.dtype);
-        return TLC_OK;
-    };
+    auto get = [&](const std::string &name, int64_t rows, int64_t cols, tlc_qtensor **t) { return bind_tensor(D, model, name, rows, cols, t); };
     const int64_t w = cfg.width;
     if (int32_t rc = get("embed", cfg.vocab, w, &D->embed)) return rc;
     if (int32_t rc = get("final.norm", 1, w, &D->final_norm)) return rc;
@@ -231,24 +171,25 @@ int32_t prepare(tlc_decoder *D) {
             }
         }
     }
-    const size_t R = (size_t)D->rows, es = D->elem, pairs = R * (size_t)std::max(D->top_max, 1);
+    // buffers of the form with one residual
+    const size_t one = cfg.streams ? 0 : 1, R = (size_t)D->rows, es = D->elem, pairs = R * (size_t)std::max(D->top_max, 1);
     D->ld_router = (int)experts_max + 1;
     struct { void **p; size_t bytes; } bufs[] = {
-        {(void **)&D->x, R * w * 4},
-        {(void **)&D->h_row, (size_t)D->ldw * 4},
-        {(void **)&D->h1, R * D->ldw * es},
-        {(void **)&D->h2, R * D->ldw * es},
-        {(void **)&D->q_raw, R * q_max * es},
-        {(void **)&D->k_raw, R * k_max * es},
-        {(void **)&D->q_rot, R * rot_max * es},
-        {(void **)&D->attn, R * attn_max * es},
-        {(void **)&D->act, R * act_max * es},
+        {(void **)&D->x, one * R * w * 4},
+        {(void **)&D->h_row, one * (size_t)D->ldw * 4},
+        {(void **)&D->h1, one * R * D->ldw * es},
+        {(void **)&D->h2, one * R * D->ldw * es},
+        {(void **)&D->q_raw, one * R * q_max * es},
+        {(void **)&D->k_raw, one * R * k_max * es},
+        {(void **)&D->q_rot, one * R * rot_max * es},
+        {(void **)&D->attn, one * R * attn_max * es},
+        {(void **)&D->act, one * R * act_max * es},
         {(void **)&D->router_out, R * D->ld_router * 4},
-        {(void **)&D->chosen, pairs * 4},
-        {(void **)&D->rank, pairs * 4},
-        {(void **)&D->place, pairs * 4},
-        {(void **)&D->weight, pairs * 4},
-        {(void **)&D->scale, pairs * 4},
+        {(void **)&D->chosen, one * pairs * 4},
+        {(void **)&D->rank, one * pairs * 4},
+        {(void **)&D->place, one * pairs * 4},
+        {(void **)&D->weight, one * pairs * 4},
+        {(void **)&D->scale, one * pairs * 4},
         {(void **)&D->count, (size_t)experts_max * 4},
         {(void **)&D->off, (size_t)(experts_max + 1) * 4},
         {(void **)&D->hp, D->top_max ? pairs * D->ldw * es : 0},
@@ -273,18 +214,16 @@ int32_t prepare(tlc_decoder *D) {
     TLC_CUDA(cudaMallocHost(&D->host_next, 64 * 4));
     TLC_CUDA(cudaMallocHost(&D->host_ids, 64 * 4));
 
+    Maps maps;
+    if (cfg.streams)
+        if (int32_t rc = prepare_streams(D, maps)) return rc;
     if (cfg.dtype != TLC_TYPE_BF16) return TLC_OK;
-    std::vector<CUtensorMap> maps;
-    int32_t bad = TLC_OK;
-    auto add = [&](const void *base, int64_t rows, int64_t cols, int64_t pitch) {
-        CUtensorMap m;
-        if (!bad) bad = encode_map(&m, base, rows, cols, pitch);
-        maps.push_back(m);
-        return (int)maps.size() - 1;
-    };
-    auto weight = [&](const tlc_qtensor *t) { return add(t->data, t->n_rows, t->n_cols, (int64_t)(t->row_pitch / 2)); };
-    D->a_h1 = add(D->h1, (int64_t)R, w, D->ldw);
-    D->a_h2 = add(D->h2, (int64_t)R, w, D->ldw);
+    auto add = [&](const void *base, int64_t rows, int64_t cols, int64_t pitch) { return maps.add(base, rows, cols, pitch); };
+    auto weight = [&](const tlc_qtensor *t) { return maps.weight(t); };
+    if (one) {
+        D->a_h1 = add(D->h1, (int64_t)R, w, D->ldw);
+        D->a_h2 = add(D->h2, (int64_t)R, w, D->ldw);
+    }
     if (D->top_max) D->a_hp = add(D->hp, (int64_t)pairs, w, D->ldw);
     D->a_hf = add(D->hf, D->logit_rows, w, D->ldw);
     D->m_embed = weight(D->embed);
@@ -308,25 +247,14 @@ int32_t prepare(tlc_decoder *D) {
             struct { const std::vector<tlc_qtensor *> &src; int *first; } fam[] = {
                 {L.e_gate, &L.m_egate}, {L.e_up, &L.m_eup}, {L.e_down, &L.m_edown}};
             for (auto &f : fam) {
-                *f.first = (int)maps.size();
+                *f.first = (int)maps.maps.size();
                 for (const tlc_qtensor *t : f.src) weight(t);
             }
         }
     }
-    if (bad) return bad;
-    return upload(D, &D->maps, maps.data(), maps.size() * sizeof(CUtensorMap));
+    if (maps.bad) return maps.bad;
+    return upload(D, &D->maps, maps.maps.data(), maps.maps.size() * sizeof(CUtensorMap));
 }
-
-// What one pass computes.
-struct Pass {
-    int m;                  // rows
-    const int *ids, *pos, *slot;
-    bool decode;            // every row is another sequence
-    int seq = 0, pos0 = 0;  // portion: its sequence and the position of row 0
-    const int *want = nullptr;  // device: rows whose logits are computed, or null: all m rows
-    int n_want = 0;
-    int want_single = -1;   // the row, when n_want == 1 and it is known on the host
-};
 
 template <typename T>
 int32_t layer_attention(tlc_decoder *D, Layer &L, int l, const Pass &ps, bool one_row) {
@@ -396,8 +324,8 @@ template <typename T>
 int32_t layers_one_row(tlc_decoder *D, const Pass &ps) {
     tlc_ctx *ctx = D->ctx;
     const int w = D->cfg.width, es = (int)sizeof(T);
-    for (int l = 0; l < D->cfg.n_layers; l++) {
-        Layer &L = D->layers[(size_t)l];
+    for (int l = 0; l < (int)D->runs.size(); l++) {
+        Layer &L = D->layers[(size_t)D->runs[(size_t)l]];
         const tlc_decoder_layer &c = L.c;
         const bool moe = c.ff_kind == TLC_FF_MOE;
         GemvParams g{};
@@ -467,44 +395,14 @@ int32_t layers_one_row(tlc_decoder *D, const Pass &ps) {
     return TLC_OK;
 }
 
-template <typename T>
-struct Gemm {  // builds one grouped launch
-    tlc_decoder *D;
-    GemmParams p{};
-    Gemm(tlc_decoder *d, int m) : D(d) {
-        p.m = m;
-        p.maps = d->maps;
-    }
-    GemmGroup &add(int n, int epi, void *out, int ldo) {
-        GemmGroup &g = p.g[p.n_groups++];
-        g = GemmGroup{};
-        g.n = n;
-        g.epi = epi;
-        g.out = out;
-        g.ldo = ldo;
-        g.b2_map = -1;
-        return g;
-    }
-    void operand(GemmGroup &g, int seg, int a_map, const void *a, int lda, int b_map, const tlc_qtensor *b) {
-        g.a_map[seg] = a_map;
-        g.a[seg] = a;
-        g.lda[seg] = lda;
-        g.b_map[seg] = b_map;
-        g.b[seg] = b->data;
-        g.ldb[seg] = (int)(b->row_pitch / sizeof(T));
-        g.k[seg] = (int)b->n_cols;
-    }
-    int32_t launch() { return launch_gemm<T>(D->ctx, p); }
-};
-
 // Many rows.  On return `pending` names the layer whose expert outputs are not in x yet, or -1.
 template <typename T>
 int32_t layers_many_rows(tlc_decoder *D, const Pass &ps, int *pending) {
     tlc_ctx *ctx = D->ctx;
     const int w = D->cfg.width, m = ps.m;
     *pending = -1;
-    for (int l = 0; l < D->cfg.n_layers; l++) {
-        Layer &L = D->layers[(size_t)l];
+    for (int l = 0; l < (int)D->runs.size(); l++) {
+        Layer &L = D->layers[(size_t)D->runs[(size_t)l]];
         const tlc_decoder_layer &c = L.c;
         const bool moe = c.ff_kind == TLC_FF_MOE;
         const int qd = c.heads * c.dim, kd = c.kv_heads * c.dim, ff = L.ff_width();
@@ -611,7 +509,7 @@ int32_t layers_many_rows(tlc_decoder *D, const Pass &ps, int *pending) {
                 GemmGroup &e = b.add(w, EPI_STORE, D->y, D->ldw);
                 b.operand(e, 0, L.a_acte, D->act_e, round8(c.expert_ff), L.m_edown, L.e_down[0]);
                 family(e, L.down_tab, nullptr);
-                *pending = l;
+                *pending = D->runs[(size_t)l];
             }
             if (int32_t rc = b.launch()) return rc;
         }
@@ -674,6 +572,7 @@ int32_t forward_t(tlc_decoder *D, const Pass &ps) {
 }
 
 int32_t forward(tlc_decoder *D, const Pass &ps) {
+    if (D->cfg.streams) return forward_streams(D, ps);
     return D->cfg.dtype == TLC_TYPE_F32 ? forward_t<float>(D, ps) : forward_t<bf16>(D, ps);
 }
 
@@ -796,17 +695,42 @@ extern "C" int32_t tlc_decoder_create(tlc_ctx *ctx, tlc_model *model, const tlc_
     D->rows = std::max(std::max(c.max_prefill, c.max_batch), 16);
     D->logit_rows = std::max(std::min(c.max_logit_rows, D->rows), c.max_batch) + 1;  // and the row that is sampled
     D->pos_hi.assign(kMaxSeqs, 0);
-    D->layers.resize((size_t)c.n_layers);
-    std::vector<int32_t> heads, dims;
-    for (int i = 0; i < c.n_layers; i++) {
-        D->layers[(size_t)i].c = c.layers[i];
-        if (int32_t rc = check_layer(c.layers[i], i)) return rc;
-        heads.push_back(c.layers[i].kv_heads);
-        dims.push_back(c.layers[i].dim);
+    TLC_REQUIRE(c.streams >= 0 && c.streams <= kMaxStreams, TLC_ERR_INVALID_DIMENSION, "decoder_create: %d residual streams (at most %d)",
+                c.streams, kMaxStreams);
+    TLC_REQUIRE(c.logit_softcap >= 0.f && (c.streams || c.logit_softcap == 0.f), TLC_ERR_INVALID_OPERATION,
+                "decoder_create: logit softcap %g", (double)c.logit_softcap);
+    TLC_REQUIRE(c.n_runs >= 0 && (c.n_runs == 0 || c.runs), TLC_ERR_INVALID_OPERATION, "decoder_create: %d runs", c.n_runs);
+    for (int r = 0; r < (c.n_runs ? c.n_runs : c.n_layers); r++) {
+        const int l = c.n_runs ? c.runs[r] : r;
+        TLC_REQUIRE(l >= 0 && l < c.n_layers, TLC_ERR_INDEX, "Index out of bounds: index %d, size %d", l, c.n_layers);
+        D->runs.push_back(l);
     }
-    D->cfg.layers = nullptr;  // the caller's array
-    if (int32_t rc = bind(D.get(), model)) return rc;
-    if (int32_t rc = tlc_kvcache_create_layers(ctx, c.dtype, c.n_layers, c.max_batch, c.max_seq, heads.data(), dims.data(), &D->cache))
+    for (int i = 0; i < c.n_layers; i++)
+        if (int32_t rc = c.streams ? check_stream_layer(c.layers[i], i) : check_layer(c.layers[i], i)) return rc;
+    std::vector<int32_t> heads, dims, latents;
+    if (c.streams) {
+        D->st.layers.resize((size_t)c.n_layers);
+        for (int i = 0; i < c.n_layers; i++) {
+            StreamLayer &L = D->st.layers[(size_t)i];
+            L.c = c.layers[i];
+            L.kp = round8(L.c.kv_rank);
+            L.row = L.kp + round8(L.c.rot_dims);
+        }
+        for (int l : D->runs) latents.push_back(D->st.layers[(size_t)l].row);
+    } else {
+        D->layers.resize((size_t)c.n_layers);
+        for (int i = 0; i < c.n_layers; i++) D->layers[(size_t)i].c = c.layers[i];
+        for (int l : D->runs) {
+            heads.push_back(c.layers[l].kv_heads);
+            dims.push_back(c.layers[l].dim);
+        }
+    }
+    D->cfg.layers = nullptr;  // the caller's arrays
+    D->cfg.runs = nullptr;
+    const int runs = (int)D->runs.size();
+    if (int32_t rc = c.streams ? bind_streams(D.get(), model) : bind(D.get(), model)) return rc;
+    if (int32_t rc = c.streams ? tlc_kvcache_create_latent(ctx, c.dtype, runs, c.max_batch, c.max_seq, latents.data(), &D->cache)
+                               : tlc_kvcache_create_layers(ctx, c.dtype, runs, c.max_batch, c.max_seq, heads.data(), dims.data(), &D->cache))
         return rc;
     if (int32_t rc = prepare(D.get())) return rc;
     TLC_CUDA(cudaFuncSetAttribute(argmax_advance_kernel<float>, cudaFuncAttributePreferredSharedMemoryCarveout,

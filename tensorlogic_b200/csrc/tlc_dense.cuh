@@ -62,6 +62,10 @@ __device__ __forceinline__ void pdl_enter() {
     pdl_trigger();
 }
 
+__device__ __forceinline__ void prefetch_l2(const void *p, uint32_t bytes) {
+    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(p), "r"(bytes) : "memory");
+}
+
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 // g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
@@ -94,9 +98,68 @@ enum Epilogue {
     EPI_STORE = 0,        // out[row][n] = T(acc [+ bias])
     EPI_STORE_F32 = 1,    // out[row][n] = acc (f32)
     EPI_ADD_F32 = 2,      // out[row][n] += acc + bias (f32: the residual stream)
-    EPI_CLAMPED_GLU = 3,  // pair: out = T(clamped_glu(gate, up) [* out_scale])
-    EPI_SILU_MUL = 4,     // pair: out = T(silu(in_scale gate) (in_scale up) [* out_scale])
+    EPI_SOFTCAP_F32 = 3,  // out[row][n] = limit * tanh(acc / limit) (f32)
+    EPI_STREAMS = 4,      // y = (acc + bias) * scale into every residual stream (StreamsOut)
+    EPI_CLAMPED_GLU = 5,  // pair: out = T(clamped_glu(gate, up) [* out_scale])
+    EPI_SILU_MUL = 6,     // pair: out = T(silu(in_scale gate [+ bias]) (in_scale up [+ bias2]) [* out_scale])
 };
+
+// ---- several residual streams (hyper-connections) -----------------------------------------------
+// The residual is n streams x_0 .. x_{n-1} (f32 planes).  A sublayer reads u = sum_s in[s] x_s through
+// its norm and leaves x_t <- sum_s mix[s][t] x_s + out[t] y.  With a norm that needs no statistics of
+// the row, tanh(alpha u) * w + b, everything behind the sublayer's last product is a function of one
+// column: the projection that makes y updates the streams and stores the NEXT sublayer's input h.
+constexpr int kMaxStreams = 8;
+struct StreamsOut {
+    float *x;               // [n][rows][width]: plane s starts at x + s * plane
+    int64_t plane;
+    int n;
+    float out[kMaxStreams], mix[kMaxStreams][kMaxStreams];  // of this sublayer; mix[from][to]
+    float in[kMaxStreams];  // of the next sublayer (all ones: the sum at the end)
+    float alpha;            // next norm
+    const void *scale;      // T [width]: multiplies y
+    const void *w, *b;      // T [width]: next norm
+    void *h;                // T [rows][ldh], or null: no next input is wanted
+    int ldh;
+};
+#ifdef __CUDACC__
+__device__ __forceinline__ float tanh_norm(float u, float alpha, float w, float b) { return tanhf(alpha * u) * w + b; }
+// One column: `x` holds the old streams and receives the new ones; returns the next sublayer's u.
+template <int MAXS>
+__device__ __forceinline__ float update_streams(const StreamsOut &o, float y, float (&x)[MAXS]) {
+    float nw[MAXS], u = 0.f;
+#pragma unroll
+    for (int t = 0; t < MAXS; t++) {
+        if (t >= o.n) break;
+        float v = o.out[t] * y;
+#pragma unroll
+        for (int s = 0; s < MAXS; s++)
+            if (s < o.n) v = fmaf(o.mix[s][t], x[s], v);
+        nw[t] = v;
+        u = fmaf(o.in[t], v, u);
+    }
+#pragma unroll
+    for (int t = 0; t < MAXS; t++)
+        if (t < o.n) x[t] = nw[t];
+    return u;
+}
+// The same with loads and stores, for column n of row `row` and the finished product `acc`.
+template <typename T>
+__device__ __forceinline__ void streams_column(const StreamsOut &o, int64_t row, int width, int n, float acc) {
+    float x[kMaxStreams];
+    float *at = o.x + row * width + n;
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; s++)
+        if (s < o.n) x[s] = __ldcg(at + s * o.plane);
+    const float u = update_streams(o, acc * to_f32(static_cast<const T *>(o.scale)[n]), x);
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; s++)
+        if (s < o.n) at[s * o.plane] = x[s];
+    if (o.h)
+        static_cast<T *>(o.h)[row * o.ldh + n] =
+            from_f32<T>(tanh_norm(u, o.alpha, to_f32(static_cast<const T *>(o.w)[n]), to_f32(static_cast<const T *>(o.b)[n])));
+}
+#endif
 
 // ---- one activation row (decode): streams weight rows -------------------------------------------
 // A segment of the output: n rows of a weight (pair: 2 n rows, gate and up alternating), all
@@ -104,6 +167,7 @@ enum Epilogue {
 struct GemvSeg {
     const void *w, *w2;  // w2: the up weight of a pair
     const void *bias;    // T [n] or null
+    const void *bias2;   // T [n] or null: of the up weight
     void *out;
     int n;               // outputs
     int v0;              // first virtual row (even)
@@ -160,6 +224,7 @@ struct OutParams {
     float *x;
     int n, pieces;            // 16-byte pieces of the whole concatenation
     int expert_split, rows_cap, prefetch;
+    StreamsOut st;            // st.n > 0: the sums go into the streams instead of x (without experts)
 };
 template <typename T>
 int32_t launch_out_gemv(tlc_ctx *ctx, OutParams &p);
@@ -176,7 +241,8 @@ struct GemmGroup {
     const void *a[2], *b[2], *b2;        // the same operands as pointers (f32 form)
     int lda[2], ldb[2], k[2];
     int n, epi;
-    const void *bias;
+    int rows, a_row0, b_row0;  // dense groups: rows of A (and out), where they start in A's map and where B's do
+    const void *bias, *bias2;  // bias2: of the up weight
     void *out;
     int ldo;
     float limit;
@@ -197,17 +263,25 @@ struct GemmParams {
     const CUtensorMap *maps;
     tlc_dev_status *status;
     uint64_t wait_ns;
+    StreamsOut st;  // of the EPI_STREAMS group (at most one)
 };
 constexpr int kMaxSlots = 1100;
 // bf16: tcgen05; f32: FMA pipes, no reduced precision.
 template <typename T>
 int32_t launch_gemm(tlc_ctx *ctx, GemmParams &p);
-// Tensor map of a row-major bf16 matrix in boxes of 128 rows x 64 columns.
-int32_t encode_map(CUtensorMap *map, const void *base, int64_t rows, int64_t cols, int64_t pitch);
+// Tensor map of a row-major bf16 matrix in boxes of `box_rows` (at most 256) rows x 64 columns.
+int32_t encode_map(CUtensorMap *map, const void *base, int64_t rows, int64_t cols, int64_t pitch, int box_rows = 128);
 
 // ---- norms, rotation, routing --------------------------------------------------------------------
 template <typename T>
 int32_t launch_embed(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int m, float *x);
+
+// Several streams: every plane of `st` gets the embedding rows; h receives norm(sum(in) * row).
+template <typename T>
+int32_t launch_embed_streams(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int m, const StreamsOut &st);
+// h[i] = norm(sum_s in[s] x_s[rows[i]]) for m rows (rows null: i itself).
+template <typename T>
+int32_t launch_streams_norm(tlc_ctx *ctx, const StreamsOut &st, int width, const int *rows, int m);
 
 // Layer norms of the rows of x; a pending sum of expert outputs is added to x first.
 struct NormParams {
@@ -293,5 +367,58 @@ int32_t launch_window_decode(tlc_ctx *ctx, WindowAttn p);
 template <typename T>
 int32_t launch_window_rows(tlc_ctx *ctx, const WindowAttn &p);
 bool window_tensor_cores(int D);
+
+// ---- latent attention ------------------------------------------------------------------------------
+// Keys and values of all heads are projections of one latent c (size KR) per token, plus one rotated key
+// part (size R) all heads share; the cache holds rows [c, 0.. | rotated part, 0..] of `row` values, the
+// rotated part at kp.  Two forms of the same scores:
+//   absorbed  q' = W_uk^T q per head, scores q'.c + q_rot.k_rot, values c, W_uv applied to the weighted
+//             latent: the cache is read once for all heads (decode, short portions, every f32 pass);
+//   expanded  keys W_uk c and values W_uv c are made for a stretch of the cache first (long portions).
+// Softmax: one more term exp(sink[head]) in the denominator.
+struct LatentParams {
+    int H, D, R, V, QR, KR;   // heads; unrotated, rotated, value size per head; query and key/value latent
+    int kp, row;              // KR padded to 8; values of a cache row
+    int m, max_seq;
+    float eps, scale;
+    const void *dq_norm, *dkv_norm, *sink;  // T
+    const void *uq, *uk, *uv;               // T, rows of *_pitch values
+    int uq_pitch, uk_pitch, uv_pitch;
+    const float *freq;        // [R / 2]
+    const void *cq_raw;       // T [m][ldcq]: W_dq h
+    const void *ckv_raw;      // T [m][ldckv]: W_dkv h
+    int ldcq, ldckv;
+    void *cq;                 // T [m][ldcq]: normalized (many rows)
+    const void *q;            // T [m][ldq]: W_uq cq (many rows; null: the query kernel makes it)
+    int ldq;
+    void *cache;              // T [slot][max_seq][row]
+    const int *pos, *slot;
+    void *ql;                 // T [m][H][row]: absorbed queries
+    float *part, *stat;       // [m][nsplit][H][kp]; [m][nsplit][H][2]: maximum (base 2) and sum
+    int nsplit;
+    void *out;                // T [m][ldo], head h at h * V
+    int ldo;
+    // expanded
+    const void *k_all;        // bf16 [keys][ldk]: unrotated keys, head h at h * D
+    const void *v_all;        // bf16 [H * V][ldv]: values, transposed
+    int ldk, ldv;
+    int pos0, slot0;          // rows are consecutive positions from pos0 of sequence slot0
+    const CUtensorMap *q_map, *k_map, *v_map, *rot_map;  // of q, k_all, v_all, the cache's rotated parts
+    tlc_dev_status *status;
+    uint64_t wait_ns;
+};
+// Many rows: latents normalized and appended to the cache, query latents normalized into cq.
+template <typename T>
+int32_t launch_latent_rows(tlc_ctx *ctx, const LatentParams &p);
+// Absorbed queries.  p.q null (one row): also the norms, W_uq and the cache append.
+template <typename T>
+int32_t launch_latent_query(tlc_ctx *ctx, const LatentParams &p);
+// Attention over the cache in p.nsplit stretches, then merge, sink and W_uv.
+template <typename T>
+int32_t launch_latent_absorbed(tlc_ctx *ctx, const LatentParams &p);
+int latent_splits(const tlc_ctx *ctx, const LatentParams &p);  // stretches for p.m rows of p.H heads
+// Expanded: attention of consecutive rows over k_all, v_all and the cache's rotated parts (bf16).
+int32_t launch_latent_prefill(tlc_ctx *ctx, const LatentParams &p);
+bool latent_prefill_fits(int D, int R, int V);
 
 }  // namespace tlc_dense

@@ -25,6 +25,9 @@ constexpr int kABytes = 128 * 128, kBBytes = 256 * 128, kStageBytesD = kABytes +
 constexpr int kEpilogueWarps = 8;  // two per lane quarter of the tensor memory, taking the column pieces in turn
 constexpr int kThreadsD = 32 * (2 + kEpilogueWarps);  // and the TMA warp, the MMA warp
 constexpr size_t kSmemD = 1024 + (size_t)kStagesD * kStageBytesD + 256 + (size_t)(2 * kMaxSlots + 4) * sizeof(int);
+constexpr int kTurnPitch = 20;  // floats per row of an epilogue warp's turning area: 32 rows of 16 columns
+constexpr size_t kSmemTurn = (size_t)kEpilogueWarps * 32 * kTurnPitch * sizeof(float);
+static_assert(((2 * kMaxSlots + 4) * sizeof(int)) % 16 == 0, "the turning area starts on a 16-byte boundary");
 
 // Instruction descriptor: bf16 x bf16 -> f32, both operands K-major, M = 128, N = 256.
 constexpr uint32_t kIdescBf16 = idesc_for(256) | (1u << 7) | (1u << 10);
@@ -48,7 +51,7 @@ __device__ void plan_tiles(const GemmParams &p, int *start, int *first_row) {
         const int nt = (gr.n + bn - 1) / bn, slots = gr.experts > 0 ? gr.experts : 1;
         for (int e = tid; e < slots; e += blockDim.x) {
             const int lo = gr.experts > 0 ? __ldcg(gr.off + e) : 0;
-            const int rows = gr.experts > 0 ? __ldcg(gr.off + e + 1) - lo : p.m;
+            const int rows = gr.experts > 0 ? __ldcg(gr.off + e + 1) - lo : gr.rows;
             start[base + e] = (rows + BM - 1) / BM * nt;
             first_row[base + e] = lo;
         }
@@ -90,7 +93,7 @@ __device__ __forceinline__ Tile tile_at(const GemmParams &p, const int *start, c
     r.expert = slot - base;
     const GemmGroup &gr = p.g[g];
     const int lo = first_row[slot];
-    const int rows = gr.experts > 0 ? __ldcg(gr.off + r.expert + 1) - lo : p.m;
+    const int rows = gr.experts > 0 ? __ldcg(gr.off + r.expert + 1) - lo : gr.rows;
     const int mt = (rows + BM - 1) / BM, local = t - start[slot];
     const int m = local % mt, n = local / mt;  // row tiles fastest: a weight tile is shared by neighbours
     r.row0 = lo + m * BM;
@@ -104,7 +107,7 @@ __device__ __forceinline__ Tile tile_at(const GemmParams &p, const int *start, c
 __device__ __forceinline__ void store_piece(const GemmGroup &g, const uint32_t (&acc)[32], const uint32_t (&up)[32], int row,
                                             int nb) {
     const bool whole = nb + 32 <= g.n;
-    if (g.epi == EPI_ADD_F32 || g.epi == EPI_STORE_F32) {
+    if (g.epi == EPI_ADD_F32 || g.epi == EPI_STORE_F32 || g.epi == EPI_SOFTCAP_F32) {
         float *out = static_cast<float *>(g.out) + (size_t)row * g.ldo + nb;
         const bool add = g.epi == EPI_ADD_F32;
         if (whole && (g.ldo & 3) == 0) {
@@ -119,14 +122,22 @@ __device__ __forceinline__ void store_piece(const GemmGroup &g, const uint32_t (
                 o.y += __uint_as_float(acc[4 * v + 1]) + b[1];
                 o.z += __uint_as_float(acc[4 * v + 2]) + b[2];
                 o.w += __uint_as_float(acc[4 * v + 3]) + b[3];
+                if (g.epi == EPI_SOFTCAP_F32) {
+                    o.x = g.limit * tanhf(o.x / g.limit);
+                    o.y = g.limit * tanhf(o.y / g.limit);
+                    o.z = g.limit * tanhf(o.z / g.limit);
+                    o.w = g.limit * tanhf(o.w / g.limit);
+                }
                 *reinterpret_cast<float4 *>(out + 4 * v) = o;
             }
         } else {
 #pragma unroll
             for (int e = 0; e < 32; e++)
-                if (nb + e < g.n)
-                    out[e] = (add ? out[e] : 0.f) + __uint_as_float(acc[e]) +
-                             (g.bias ? to_f32(static_cast<const bf16 *>(g.bias)[nb + e]) : 0.f);
+                if (nb + e < g.n) {
+                    const float v = (add ? out[e] : 0.f) + __uint_as_float(acc[e]) +
+                                    (g.bias ? to_f32(static_cast<const bf16 *>(g.bias)[nb + e]) : 0.f);
+                    out[e] = g.epi == EPI_SOFTCAP_F32 ? g.limit * tanhf(v / g.limit) : v;
+                }
         }
         return;
     }
@@ -147,8 +158,14 @@ __device__ __forceinline__ void store_piece(const GemmGroup &g, const uint32_t (
                 h[e] = from_f32<bf16>(clamped_glu(si * __uint_as_float(acc[e]), si * __uint_as_float(up[e]), g.limit) * so);
         } else {
 #pragma unroll
-            for (int e = 0; e < 32; e++)
-                h[e] = from_f32<bf16>(silu_mul(si * __uint_as_float(acc[e]), si * __uint_as_float(up[e])) * so);
+            for (int e = 0; e < 32; e++) {
+                float gate = si * __uint_as_float(acc[e]), u = si * __uint_as_float(up[e]);
+                if (g.bias && (whole || nb + e < g.n)) {
+                    gate += to_f32(static_cast<const bf16 *>(g.bias)[nb + e]);
+                    u += to_f32(static_cast<const bf16 *>(g.bias2)[nb + e]);
+                }
+                h[e] = from_f32<bf16>(silu_mul(gate, u) * so);
+            }
         }
     }
     bf16 *out = static_cast<bf16 *>(g.out) + (size_t)row * g.ldo + nb;
@@ -162,6 +179,95 @@ __device__ __forceinline__ void store_piece(const GemmGroup &g, const uint32_t (
     }
 }
 
+// 32 columns of the warp's 32 rows (lane = row of `acc`) into the residual streams.  Rows turn into
+// columns through shared memory, 16 columns at a time, so that four lanes share a row's 64 bytes and
+// the loads of all streams are in flight together.  The first `rows` of the 32 exist.
+template <int MAXS>
+__device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsOut &st, const uint32_t (&acc)[32], float *turn,
+                                              int row0, int rows, int nb, int lane) {
+#pragma unroll
+    for (int half = 0; half < 2; half++) {
+        if (nb + 16 * half >= g.n) break;
+        __syncwarp();
+#pragma unroll
+        for (int v = 0; v < 4; v++)
+            *reinterpret_cast<float4 *>(turn + lane * kTurnPitch + 4 * v) =
+                make_float4(__uint_as_float(acc[16 * half + 4 * v]), __uint_as_float(acc[16 * half + 4 * v + 1]),
+                            __uint_as_float(acc[16 * half + 4 * v + 2]), __uint_as_float(acc[16 * half + 4 * v + 3]));
+        __syncwarp();
+        const int n = nb + 16 * half + 4 * (lane & 3);
+        if (n >= g.n) continue;
+        if ((g.n & 3) != 0) {  // rows do not start on 16-byte boundaries
+            for (int i = lane >> 2; i < rows; i += 8)
+                for (int e = 0; e < 4 && n + e < g.n; e++)
+                    streams_column<bf16>(st, row0 + i, g.n, n + e,
+                                         turn[i * kTurnPitch + 4 * (lane & 3) + e] +
+                                             (g.bias ? to_f32(static_cast<const bf16 *>(g.bias)[n + e]) : 0.f));
+            continue;
+        }
+        auto four = [&](const void *p, float (&f)[4]) {
+            const uint2 v = __ldg(reinterpret_cast<const uint2 *>(static_cast<const bf16 *>(p) + n));
+            f[0] = __uint_as_float(v.x << 16);
+            f[1] = __uint_as_float(v.x & 0xffff0000u);
+            f[2] = __uint_as_float(v.y << 16);
+            f[3] = __uint_as_float(v.y & 0xffff0000u);
+        };
+        float bias[4] = {0.f, 0.f, 0.f, 0.f}, scale[4], w[4], b[4];
+        if (g.bias) four(g.bias, bias);
+        four(st.scale, scale);
+        if (st.h) {
+            four(st.w, w);
+            four(st.b, b);
+        }
+        constexpr int AT_ONCE = MAXS > 4 ? 2 : 4;
+#pragma unroll
+        for (int i0 = 0; i0 < 4; i0 += AT_ONCE) {
+            float4 x[AT_ONCE][MAXS];
+#pragma unroll
+            for (int i = 0; i < AT_ONCE; i++) {
+                const int r = 8 * (i0 + i) + (lane >> 2);
+#pragma unroll
+                for (int s = 0; s < MAXS; s++)
+                    if (s < st.n && r < rows)
+                        x[i][s] = __ldcg(reinterpret_cast<const float4 *>(st.x + s * st.plane + (int64_t)(row0 + r) * g.n + n));
+            }
+#pragma unroll
+            for (int i = 0; i < AT_ONCE; i++) {
+                const int r = 8 * (i0 + i) + (lane >> 2);
+                if (r >= rows) continue;
+                const float4 a = *reinterpret_cast<const float4 *>(turn + r * kTurnPitch + 4 * (lane & 3));
+                const float av[4] = {a.x, a.y, a.z, a.w};
+                float h[4];
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    float xs[MAXS];
+#pragma unroll
+                    for (int s = 0; s < MAXS; s++) xs[s] = e == 0 ? x[i][s].x : e == 1 ? x[i][s].y : e == 2 ? x[i][s].z : x[i][s].w;
+                    const float u = update_streams(st, (av[e] + bias[e]) * scale[e], xs);
+#pragma unroll
+                    for (int s = 0; s < MAXS; s++) {
+                        if (e == 0) x[i][s].x = xs[s];
+                        if (e == 1) x[i][s].y = xs[s];
+                        if (e == 2) x[i][s].z = xs[s];
+                        if (e == 3) x[i][s].w = xs[s];
+                    }
+                    h[e] = st.h ? tanh_norm(u, st.alpha, w[e], b[e]) : 0.f;
+                }
+#pragma unroll
+                for (int s = 0; s < MAXS; s++)
+                    if (s < st.n) *reinterpret_cast<float4 *>(st.x + s * st.plane + (int64_t)(row0 + r) * g.n + n) = x[i][s];
+                if (st.h) {
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(h[0], h[1]), hi = __floats2bfloat162_rn(h[2], h[3]);
+                    *reinterpret_cast<uint2 *>(static_cast<bf16 *>(st.h) + (int64_t)(row0 + r) * st.ldh + n) =
+                        make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+                }
+            }
+        }
+    }
+}
+
+// MAXS > 0: the form whose groups end in EPI_STREAMS, for up to MAXS streams.
+template <int MAXS>
 __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t *tiles = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -171,6 +277,7 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
     volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
     int *start = reinterpret_cast<int *>(reinterpret_cast<uint8_t *>(full) + 256);
     int *first_row = start + kMaxSlots + 2;
+    [[maybe_unused]] float *turning = reinterpret_cast<float *>(first_row + kMaxSlots + 2);
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (tid == 0) {
@@ -210,7 +317,7 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
                     const CUtensorMap *am = p.maps + g.a_map[seg];
                     const CUtensorMap *bm = p.maps + g.b_map[seg] + (size_t)tl.expert * g.map_stride;
                     const CUtensorMap *um = g.b2_map >= 0 ? p.maps + g.b2_map + (size_t)tl.expert * g.map_stride : bm;
-                    const int second = g.b2_map >= 0 ? tl.n0 : tl.n0 + 128;  // rows of the tile's upper half
+                    const int first = g.b_row0 + tl.n0, second = g.b2_map >= 0 ? first : first + 128;  // rows of the tile's halves
                     for (int s = 0; s < steps; s++, j++) {
                         const int st = j % kStagesD;
                         if (!mbar_wait(&empty[st], ((j / kStagesD) & 1u) ^ 1u, abort_flag, p.status, 21, p.wait_ns)) {
@@ -220,8 +327,8 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
                         const uint32_t bar = smem_u32(&full[st]);
                         const uint32_t at = smem_u32(tiles + (size_t)st * kStageBytesD);
                         mbar_arrive_expect_tx(&full[st], kStageBytesD);
-                        tma_load_2d(at, am, s * kBK, tl.row0, bar);
-                        tma_load_2d(at + kABytes, bm, s * kBK, tl.n0, bar);
+                        tma_load_2d(at, am, s * kBK, g.a_row0 + tl.row0, bar);
+                        tma_load_2d(at + kABytes, bm, s * kBK, first, bar);
                         tma_load_2d(at + kABytes + 128 * 128, um, s * kBK, second, bar);
                     }
                 }
@@ -274,7 +381,13 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
                 const uint32_t at = tmem + ((uint32_t)(32 * wq) << 16) + 256 * a + 32 * c;
                 tmem_ld32(at, r);
                 if (pair) tmem_ld32(at + 128, u);
-                if (done && row < tl.rows) store_piece(g, r, u, tl.row0 + row, tl.n0 + 32 * c);
+                if constexpr (MAXS > 0) {
+                    if (done && g.epi == EPI_STREAMS)
+                        store_streams<MAXS>(g, p.st, r, turning + (warp - 2) * 32 * kTurnPitch, tl.row0 + 32 * wq, tl.rows - 32 * wq,
+                                            tl.n0 + 32 * c, lane);
+                } else {
+                    if (done && row < tl.rows) store_piece(g, r, u, tl.row0 + row, tl.n0 + 32 * c);
+                }
             }
             tc_fence_before();
             __syncwarp();
@@ -350,11 +463,18 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const __grid_consta
                 float *out = static_cast<float *>(g.out) + (size_t)row * g.ldo + n;
                 float v = acc[i][j];
                 if (pair) {
-                    v = g.epi == EPI_CLAMPED_GLU ? clamped_glu(si * v, si * acu[i][j], g.limit) : silu_mul(si * v, si * acu[i][j]);
-                    v *= so;
+                    float gate = si * v, up = si * acu[i][j];
+                    if (g.bias) gate += static_cast<const float *>(g.bias)[n];
+                    if (g.bias2) up += static_cast<const float *>(g.bias2)[n];
+                    v = (g.epi == EPI_CLAMPED_GLU ? clamped_glu(gate, up, g.limit) : silu_mul(gate, up)) * so;
                 } else {
                     if (g.bias) v += static_cast<const float *>(g.bias)[n];
+                    if (g.epi == EPI_STREAMS) {
+                        streams_column<float>(p.st, row, g.n, n, v);
+                        continue;
+                    }
                     if (g.epi == EPI_ADD_F32) v += *out;
+                    if (g.epi == EPI_SOFTCAP_F32) v = g.limit * tanhf(v / g.limit);
                 }
                 *out = v;
             }
@@ -373,7 +493,7 @@ long tile_bound(const GemmParams &p, int bm, int bn_single, int bn_pair, const i
             const long used = rows < p.g[g].experts ? rows : p.g[g].experts;
             t += nt * (used + rows / bm);
         } else {
-            t += nt * ((p.m + bm - 1) / bm);
+            t += nt * ((p.g[g].rows + bm - 1) / bm);
         }
     }
     return t;
@@ -381,7 +501,7 @@ long tile_bound(const GemmParams &p, int bm, int bn_single, int bn_pair, const i
 
 }  // namespace
 
-int32_t encode_map(CUtensorMap *map, const void *base, int64_t rows, int64_t cols, int64_t pitch) {
+int32_t encode_map(CUtensorMap *map, const void *base, int64_t rows, int64_t cols, int64_t pitch, int box_rows) {
     static PFN_cuTensorMapEncodeTiled_v12000 encode = [] {
         void *fn = nullptr;
         cudaDriverEntryPointQueryResult qres;
@@ -396,7 +516,7 @@ int32_t encode_map(CUtensorMap *map, const void *base, int64_t rows, int64_t col
                 "tensor map: base and rows must be 16-byte aligned");
     const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
     const cuuint64_t strides[1] = {(cuuint64_t)pitch * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)kBK, 128};
+    const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)box_rows};
     const cuuint32_t estr[2] = {1, 1};
     const CUresult rc = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
                                CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -412,27 +532,34 @@ static int32_t count_slots(GemmParams &p) {
     return TLC_OK;
 }
 
-template <>
-int32_t launch_gemm<bf16>(tlc_ctx *ctx, GemmParams &p) {
-    if (int32_t rc = count_slots(p)) return rc;
+template <int MAXS>
+static int32_t launch_tensor(tlc_ctx *ctx, const GemmParams &p, long ctas) {
     static bool done[64] = {};
+    constexpr size_t smem = kSmemD + (MAXS > 0 ? kSmemTurn : 0);
     if (!done[ctx->device & 63]) {
-        TLC_CUDA(cudaFuncSetAttribute(dense_gemm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemD));
+        TLC_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<MAXS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         done[ctx->device & 63] = true;
     }
-    p.status = ctx->dev_status;
-    p.wait_ns = ctx->wait_ns;
-    int family[6];
-    for (int g = 0; g < p.n_groups; g++) family[g] = p.g[g].experts > 0 ? p.m * p.g[g].in_rows_per_token : 0;
-    long tiles = tile_bound(p, 128, 256, 128, family);
-    if (tiles > ctx->sm_count) tiles = ctx->sm_count;
-    cudaError_t le = tlc_launch_pdl(ctx, dense_gemm_kernel, dim3((unsigned)tiles), dim3(kThreadsD), kSmemD, p);
+    cudaError_t le = tlc_launch_pdl(ctx, dense_gemm_kernel<MAXS>, dim3((unsigned)ctas), dim3(kThreadsD), smem, p);
     if (le != cudaSuccess) {
         cudaGetLastError();
         return tlc_fail(TLC_ERR_CUDA, "dense gemm launch failed: %s", cudaGetErrorString(le));
     }
     TLC_CHECK_LAUNCH(ctx);
     return TLC_OK;
+}
+
+template <>
+int32_t launch_gemm<bf16>(tlc_ctx *ctx, GemmParams &p) {
+    if (int32_t rc = count_slots(p)) return rc;
+    p.status = ctx->dev_status;
+    p.wait_ns = ctx->wait_ns;
+    int family[6];
+    for (int g = 0; g < p.n_groups; g++) family[g] = p.g[g].experts > 0 ? p.m * p.g[g].in_rows_per_token : 0;
+    long tiles = tile_bound(p, 128, 256, 128, family);
+    if (tiles > ctx->sm_count) tiles = ctx->sm_count;
+    if (p.st.n == 0) return launch_tensor<0>(ctx, p, tiles);
+    return p.st.n <= 4 ? launch_tensor<4>(ctx, p, tiles) : launch_tensor<kMaxStreams>(ctx, p, tiles);
 }
 
 template <>

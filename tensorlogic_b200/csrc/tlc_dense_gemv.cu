@@ -79,9 +79,6 @@ __device__ __forceinline__ uint4 load_weight(const uint4 *p) {
                  : "l"(p));
     return v;
 }
-__device__ __forceinline__ void prefetch_l2(const void *p, uint32_t bytes) {
-    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(p), "r"(bytes) : "memory");
-}
 
 template <typename T>
 __device__ __forceinline__ float dot_piece(const uint4 &w, const float *plane0, const float *plane1, int c) {
@@ -293,13 +290,16 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const __grid_constant
         const int j = v - g.v0;
         if (g.w2) {
             if (j & 1) continue;
-            const float gate = total(r), up = total(r + 1);
+            float gate = total(r), up = total(r + 1);
+            if (g.bias) gate += to_f32(static_cast<const T *>(g.bias)[j >> 1]);
+            if (g.bias2) up += to_f32(static_cast<const T *>(g.bias2)[j >> 1]);
             static_cast<T *>(g.out)[j >> 1] =
                 from_f32<T>(g.epi == EPI_CLAMPED_GLU ? clamped_glu(gate, up, g.limit) : silu_mul(gate, up));
         } else if (j < g.n) {
             float a = total(r);
             if (g.bias) a += to_f32(static_cast<const T *>(g.bias)[j]);
-            if (g.epi == EPI_STORE_F32)
+            if (g.epi == EPI_SOFTCAP_F32) a = g.limit * tanhf(a / g.limit);
+            if (g.epi == EPI_STORE_F32 || g.epi == EPI_SOFTCAP_F32)
                 static_cast<float *>(g.out)[j] = a;
             else
                 static_cast<T *>(g.out)[j] = from_f32<T>(a);
@@ -479,7 +479,10 @@ __global__ void __launch_bounds__(kThreads, 2) out_gemv_kernel(const __grid_cons
         for (int i = 0; i < slots; i++) a += part[r * slots + i];
         const int n = r_lo + r;
         if (p.bias) a += to_f32(static_cast<const T *>(p.bias)[n]);
-        p.x[n] = __ldcg(p.x + n) + a;
+        if (p.st.n > 0)
+            streams_column<T>(p.st, 0, p.n, n, a);
+        else
+            p.x[n] = __ldcg(p.x + n) + a;
     }
 }
 

@@ -140,6 +140,59 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const NormParams p) {
     }
 }
 
+// Embedding rows into every residual stream, and the first sublayer's input.
+template <typename T>
+__global__ void embed_streams_kernel(const T *__restrict__ table, int64_t pitch, int vocab, int d, const int *__restrict__ ids,
+                                     const __grid_constant__ StreamsOut st) {
+    constexpr int N = Vec<T>::N;
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * N, r = blockIdx.y;
+    float w[N], b[N];
+    if (i < d) {  // weights: rows are padded to whole pieces
+        unpack(__ldg(reinterpret_cast<const uint4 *>(static_cast<const T *>(st.w) + i)), w);
+        unpack(__ldg(reinterpret_cast<const uint4 *>(static_cast<const T *>(st.b) + i)), b);
+    }
+    pdl_enter();  // ids are written by the previous step's sampling kernel
+    if (i >= d) return;
+    int id = ids[r];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; never read outside
+    float f[N], sum = 0.f;
+    unpack(__ldg(reinterpret_cast<const uint4 *>(table + (size_t)id * pitch + i)), f);
+    for (int s = 0; s < st.n; s++) sum += st.in[s];
+    float *x = st.x + (size_t)r * d + i;
+    T *h = static_cast<T *>(st.h) + (size_t)r * st.ldh + i;
+    if ((d & 3) == 0 && i + N <= d) {
+        for (int s = 0; s < st.n; s++)
+#pragma unroll
+            for (int e = 0; e < N; e += 4)
+                *reinterpret_cast<float4 *>(x + s * st.plane + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+#pragma unroll
+        for (int e = 0; e < N; e += 4) {
+            float v[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) v[j] = tanh_norm(sum * f[e + j], st.alpha, w[e + j], b[e + j]);
+            store4(h + e, v);
+        }
+    } else {
+#pragma unroll
+        for (int e = 0; e < N; e++)
+            if (i + e < d) {
+                for (int s = 0; s < st.n; s++) x[s * st.plane + e] = f[e];
+                h[e] = from_f32<T>(tanh_norm(sum * f[e], st.alpha, w[e], b[e]));
+            }
+    }
+}
+
+template <typename T>
+__global__ void streams_norm_kernel(const __grid_constant__ StreamsOut st, int d, const int *__restrict__ rows) {
+    pdl_enter();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x, src = rows ? rows[blockIdx.y] : blockIdx.y;
+    if (i >= d) return;
+    float u = 0.f;
+    for (int s = 0; s < st.n; s++) u = fmaf(st.in[s], __ldcg(st.x + s * st.plane + (size_t)src * d + i), u);
+    static_cast<T *>(st.h)[(size_t)blockIdx.y * st.ldh + i] =
+        from_f32<T>(tanh_norm(u, st.alpha, to_f32(static_cast<const T *>(st.w)[i]), to_f32(static_cast<const T *>(st.b)[i])));
+}
+
 // One CTA per row: RMS norm of all query heads at once and of all key heads at once, rotation of
 // the first `rot` values of every head, queries to q_out, keys and raw keys (= values) to the cache.
 template <typename T>
@@ -352,6 +405,22 @@ int32_t launch_embed(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int
 }
 
 template <typename T>
+int32_t launch_embed_streams(tlc_ctx *ctx, const tlc_qtensor *table, const int *ids, int m, const StreamsOut &st) {
+    const int d = (int)table->n_cols, threads = 128, per = (d + threads * Vec<T>::N - 1) / (threads * Vec<T>::N);
+    cudaError_t le = tlc_launch_pdl(ctx, embed_streams_kernel<T>, dim3(per, m), dim3(threads), 0, static_cast<const T *>(table->data),
+                                    (int64_t)(table->row_pitch / sizeof(T)), (int)table->n_rows, d, ids, st);
+    TLC_LAUNCHED(ctx, le, "embedding");
+    return TLC_OK;
+}
+
+template <typename T>
+int32_t launch_streams_norm(tlc_ctx *ctx, const StreamsOut &st, int width, const int *rows, int m) {
+    cudaError_t le = tlc_launch_pdl(ctx, streams_norm_kernel<T>, dim3((width + 255) / 256, m), dim3(256), 0, st, width, rows);
+    TLC_LAUNCHED(ctx, le, "streams norm");
+    return TLC_OK;
+}
+
+template <typename T>
 int32_t launch_norm(tlc_ctx *ctx, const NormParams &p) {
     const size_t smem = (size_t)p.d * sizeof(float);
     static bool done[64] = {};
@@ -394,6 +463,10 @@ int32_t launch_permute(tlc_ctx *ctx, const PermuteParams &p) {
 
 template int32_t launch_embed<bf16>(tlc_ctx *, const tlc_qtensor *, const int *, int, float *);
 template int32_t launch_embed<float>(tlc_ctx *, const tlc_qtensor *, const int *, int, float *);
+template int32_t launch_embed_streams<bf16>(tlc_ctx *, const tlc_qtensor *, const int *, int, const StreamsOut &);
+template int32_t launch_embed_streams<float>(tlc_ctx *, const tlc_qtensor *, const int *, int, const StreamsOut &);
+template int32_t launch_streams_norm<bf16>(tlc_ctx *, const StreamsOut &, int, const int *, int);
+template int32_t launch_streams_norm<float>(tlc_ctx *, const StreamsOut &, int, const int *, int);
 template int32_t launch_norm<bf16>(tlc_ctx *, const NormParams &);
 template int32_t launch_norm<float>(tlc_ctx *, const NormParams &);
 template int32_t launch_qk_rotate<bf16>(tlc_ctx *, const RotParams &, int);

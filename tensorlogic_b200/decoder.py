@@ -1,6 +1,7 @@
 """Config-driven decoder: dense bf16 / f32 weights, layers described one by one.
 
-    DecoderArch / LayerArch   sizes and constants of a model, read by its design's module
+    DecoderArch / LayerArch / LatentLayerArch
+                              sizes and constants of a model, read by its design's module
     Decoder                   the runner (tlc_decoder_* of include/tlcuda.h): sequences with cache
                               slots, portions of prompts, greedy or temperature decoding
     load_safetensors          a safetensors file -> Model
@@ -47,7 +48,69 @@ class LayerArch:
         kind = {"none": _lib.FF_NONE, "clamped_glu": _lib.FF_CLAMPED_GLU, "moe": _lib.FF_MOE}[self.ff_kind]
         return DecoderLayer(self.heads, self.kv_heads, self.dim, min(self.window, 2**31 - 1), self.keep_first, self.rot_dims,
                             self.rot_base, self.scale, kind, self.ff, self.limit, self.experts, self.top, self.expert_ff,
-                            self.shared_ff)
+                            self.shared_ff, _lib.MIX_WINDOW)
+
+    def tensor_shapes(self, p: str, w: int, _streams: int) -> dict:
+        q, k = self.heads * self.dim, self.kv_heads * self.dim
+        out = {p + "norm1": (1, w), p + "mix.q": (q, w), p + "mix.q.b": (1, q), p + "mix.q.norm": (1, q), p + "mix.k": (k, w),
+               p + "mix.k.b": (1, k), p + "mix.k.norm": (1, k), p + "mix.o": (w, q), p + "mix.o.b": (1, w)}
+        if self.ff_kind != "none":
+            out[p + "norm2"] = (1, w)
+
+        def glu(at, n):
+            out.update({at + "gate": (n, w), at + "up": (n, w), at + "down": (w, n)})
+        if self.ff_kind == "clamped_glu":
+            glu(p + "mlp.", self.ff)
+        elif self.ff_kind == "moe":
+            out[p + "mlp.router"] = (self.experts, w)
+            for e in range(self.experts):
+                glu(f"{p}mlp.e{e}.", self.expert_ff)
+            if self.shared_ff:
+                glu(p + "mlp.shared.", self.shared_ff)
+                out[p + "mlp.shared.sg"] = (1, w)
+        return out
+
+
+@dataclass
+class LatentLayerArch:
+    """One layer over several residual streams: latent attention (``dim`` unrotated and ``rot_dim`` rotated
+    entries per head and key, ``vdim`` per value) and a feed-forward (``ff_kind``: "none" or "silu_glu")."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    rot_base: float
+    scale: float
+    ff_kind: str = "none"
+    ff: int = 0
+
+    def struct(self) -> DecoderLayer:
+        kind = {"none": _lib.FF_NONE, "silu_glu": _lib.FF_SILU_GLU}[self.ff_kind]
+        return DecoderLayer(heads=self.heads, dim=self.dim, rot_dims=self.rot_dim, rot_base=self.rot_base, scale=self.scale,
+                            ff_kind=kind, ff=self.ff, mixer=_lib.MIX_LATENT, vdim=self.vdim, q_rank=self.q_rank, kv_rank=self.kv_rank)
+
+    def tensor_shapes(self, p: str, w: int, streams: int) -> dict:
+        h, m = self.heads, p + "mix."
+        out = {m + "dq": (self.q_rank, w), m + "dq.norm": (1, self.q_rank), m + "uq": (h * (self.dim + self.rot_dim), self.q_rank),
+               m + "dkv": (self.kv_rank + self.rot_dim, w), m + "dkv.norm": (1, self.kv_rank), m + "uk": (h * self.dim, self.kv_rank),
+               m + "uv": (h * self.vdim, self.kv_rank), m + "sink": (1, h), m + "o": (w, h * self.vdim)}
+        for q in (1, 2) if self.ff_kind != "none" else (1,):
+            out.update({f"{p}norm{q}": (1, w), f"{p}norm{q}.b": (1, w), f"{p}norm{q}.alpha": (1, 1), f"{p}ls{q}": (1, w),
+                        f"{p}hc{q}.in": (1, streams), f"{p}hc{q}.out": (1, streams), f"{p}hc{q}.mix": (streams, streams)})
+        if self.ff_kind != "none":
+            f = p + "mlp."
+            out.update({f + "gate": (self.ff, w), f + "gate.b": (1, self.ff), f + "up": (self.ff, w), f + "up.b": (1, self.ff),
+                        f + "down": (w, self.ff), f + "down.b": (1, w)})
+        return out
+
+    def weight_bytes(self, w: int, elem: int = 2) -> int:
+        """Bytes of the matrices one token uses."""
+        h = self.heads
+        n = self.q_rank * (w + h * (self.dim + self.rot_dim)) + w * (self.kv_rank + self.rot_dim) + \
+            h * (self.dim + self.vdim) * self.kv_rank + w * h * self.vdim + (3 * w * self.ff if self.ff_kind != "none" else 0)
+        return n * elem
 
 
 @dataclass
@@ -55,35 +118,24 @@ class DecoderArch:
     width: int
     vocab: int
     norm_eps: float
-    layers: list[LayerArch] = field(default_factory=list)
+    layers: list = field(default_factory=list)   # LayerArch, or LatentLayerArch with streams > 0
+    streams: int = 0                             # residual streams; 0: one residual, parallel branches
+    logit_softcap: float = 0.0
+    runs: Optional[list[int]] = None             # layer numbers in the order they run (None: each once)
 
     def tensor_shapes(self) -> dict:
         """Tensor names -> (rows, cols) as tlc_decoder_create binds them."""
-        w = self.width
-        out = {"embed": (self.vocab, w), "final.norm": (1, w)}
+        out = {"embed": (self.vocab, self.width), "final.norm": (1, self.width)}
+        if self.streams:
+            out.update({"final.norm.b": (1, self.width), "final.norm.alpha": (1, 1)})
         for i, l in enumerate(self.layers):
-            p, q, k = f"l{i}.", l.heads * l.dim, l.kv_heads * l.dim
-            out.update({p + "norm1": (1, w), p + "mix.q": (q, w), p + "mix.q.b": (1, q), p + "mix.q.norm": (1, q),
-                        p + "mix.k": (k, w), p + "mix.k.b": (1, k), p + "mix.k.norm": (1, k), p + "mix.o": (w, q),
-                        p + "mix.o.b": (1, w)})
-            if l.ff_kind != "none":
-                out[p + "norm2"] = (1, w)
-
-            def glu(at, n):
-                out.update({at + "gate": (n, w), at + "up": (n, w), at + "down": (w, n)})
-            if l.ff_kind == "clamped_glu":
-                glu(p + "mlp.", l.ff)
-            elif l.ff_kind == "moe":
-                out[p + "mlp.router"] = (l.experts, w)
-                for e in range(l.experts):
-                    glu(f"{p}mlp.e{e}.", l.expert_ff)
-                if l.shared_ff:
-                    glu(p + "mlp.shared.", l.shared_ff)
-                    out[p + "mlp.shared.sg"] = (1, w)
+            out.update(l.tensor_shapes(f"l{i}.", self.width, self.streams))
         return out
 
-    def layer_weight_bytes(self, l: LayerArch, elem: int = 2, active_only: bool = True) -> int:
+    def layer_weight_bytes(self, l, elem: int = 2, active_only: bool = True) -> int:
         """Bytes of the matrices one token uses in layer ``l`` (all experts with active_only=False)."""
+        if isinstance(l, LatentLayerArch):
+            return l.weight_bytes(self.width, elem)
         w, q, k = self.width, l.heads * l.dim, l.kv_heads * l.dim
         n = w * (q + k) + q * w
         if l.ff_kind == "clamped_glu":
@@ -117,10 +169,14 @@ def model_from_arrays(dev: Device, weights: dict, dtype: str = "bfloat16") -> Mo
 
 
 def synthetic_decoder(dev: Device, arch: DecoderArch, seed: int, dtype: str = "bfloat16") -> Model:
-    """Random weights made on the device: matrices N(0, 1/columns), norm weights N(1, 0.02), biases N(0, 0.02)."""
+    """Random weights made on the device: matrices N(0, 1/columns), norm weights and scales N(1, 0.02), biases
+    N(0, 0.02), coefficients of n streams N(1 / n, 0.02)."""
     m = Model(dev)
     for name, (rows, cols) in arch.tensor_shapes().items():
-        mean, std = (1.0, 0.02) if "norm" in name else (0.0, 0.02) if name.endswith(".b") else (0.0, cols ** -0.5)
+        last = name.rsplit(".", 1)[-1]
+        mean, std = ((1.0 / cols, 0.02) if last in ("alpha", "mix", "in", "out") else
+                     (0.0, 0.02) if last in ("b", "sink") else (1.0, 0.02) if "norm" in name or last in ("ls1", "ls2") else
+                     (0.0, cols ** -0.5))
         h = C.c_void_p()
         check(dev.lib.tlc_qtensor_create_normal_dense(dev.handle, DTYPES[dtype], rows, cols, seed, synth.tensor_id(name), mean,
                                                       std, C.byref(h)))
@@ -146,8 +202,10 @@ class Decoder:
         if max_logit_rows is None:  # up to 256 MiB of logits
             max_logit_rows = max(1, min(max_prefill, (256 << 20) // (4 * arch.vocab)))
         layers = (DecoderLayer * len(arch.layers))(*[l.struct() for l in arch.layers])
+        runs = np.ascontiguousarray(arch.runs if arch.runs is not None else range(len(arch.layers)), np.int32)
         cfg = DecoderConfig(len(arch.layers), arch.width, arch.vocab, arch.norm_eps, DTYPES[dtype], max_seq, max_batch,
-                            max_prefill, max_logit_rows, int(not use_graph), layers)
+                            max_prefill, max_logit_rows, int(not use_graph), arch.streams, arch.logit_softcap,
+                            runs.size, layers, _ints(runs))
         h = C.c_void_p()
         check(dev.lib.tlc_decoder_create(dev.handle, model.handle, C.byref(cfg), C.byref(h)))
         self.handle = h

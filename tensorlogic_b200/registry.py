@@ -13,7 +13,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable, Iterator, Sequence
 
-from . import decoder, toposun
+from . import decoder, suselorn, toposun
 from ._lib import ERR_LOAD, TensorError
 from .api import Device
 from .model import Llama, LlamaArch, load_model
@@ -43,6 +43,7 @@ def _decoder(read_config) -> Callable[..., object]:
 ARCHITECTURES: dict[str, Entry] = {
     "llama": Entry(("float16",), _llama),
     toposun.NAME: Entry(decoder.Decoder.dtypes, _decoder(toposun.read_config), "decoder"),
+    suselorn.NAME: Entry(decoder.Decoder.dtypes, _decoder(suselorn.read_config), "decoder"),
 }
 
 
