@@ -1,11 +1,358 @@
-// Latent attention, expanded form for long portions: not there yet, every portion takes the absorbed form.
+// Latent attention, expanded form: consecutive rows of one sequence against keys and values made from the
+// cache's latents for the whole stretch (bf16, tcgen05).
+//
+// One CTA takes 128 queries of one head.  Keys come in tiles of 64: unrotated parts from k_all, the
+// rotated part all heads share straight from the cache, values transposed (V rows of 64 keys), so that
+// every operand is K-major; all by TMA with the 128-byte swizzle, two stages.
+//   warp 0       TMA
+//   warp 1       issues the MMAs: S = Q K^T of tile j + 1 before P V of tile j
+//   warps 2-9    two softmax groups of 128 threads, one query row per thread; group g owns the tiles
+//                j = g (mod 2), its own half of the scores, its own P buffer and its own accumulator,
+//                maximum and sum, so the groups never wait for one another before the end.
+// A group's accumulator is rescaled only when a row's maximum has grown by more than 2^8; weights are
+// relative to the maximum of the last rescaling, so they stay below 2^8.  A weight enters the P.V product
+// as the sum of two bf16 numbers.  At the end the two accumulators and the sink are merged.
+// All waits are bounded; a wait that runs out sets the status word and lets the CTA drain, free its tensor
+// memory and return.
 #include "tlc_dense.cuh"
+#include "tlc_gemm_kernel.cuh"
+#include "tlc_mma.cuh"
 
 namespace tlc_dense {
 
-bool latent_prefill_fits(int, int, int) { return false; }
-int32_t launch_latent_prefill(tlc_ctx *, const LatentParams &) {
-    return tlc_fail(TLC_ERR_INVALID_OPERATION, "latent attention: no expanded form");
+namespace {
+
+using tlc_gemm::fence_async_proxy;
+using tlc_gemm::make_desc;
+using tlc_gemm::mbar_arrive;
+using tlc_gemm::mbar_arrive_expect_tx;
+using tlc_gemm::mbar_init;
+using tlc_gemm::mbar_wait;
+using tlc_gemm::smem_u32;
+using tlc_gemm::tc_fence_after;
+using tlc_gemm::tc_fence_before;
+using tlc_gemm::tma_load_2d;
+using tlc_gemm::tmem_ld32;
+using tlc_gemm::umma_commit;
+using tlc_gemm::umma_f16;
+
+constexpr int kRows = 128, kTile = 64;
+constexpr int kGroup = 128, kThreadsP = 64 + 2 * kGroup;
+constexpr int kQChunk = kRows * 128, kKChunk = kTile * 128;  // bytes of 64 columns
+constexpr int kPBytes = kRows * 128;                         // one part (high or low) of a group's weights
+constexpr uint32_t kIdesc = (1u << 7) | (1u << 10);          // bf16 x bf16
+constexpr float kLog2e = 1.44269504088896340736f;
+
+struct Layout {  // of the shared memory, in bytes from a 1024-byte boundary
+    int chunks_d, chunks_r, v_rows;
+    size_t k_stage, v_stage, q, k, v, p, bars, total;
+    __host__ __device__ Layout(int D, int R, int V)
+        : chunks_d((D + 63) / 64), chunks_r((R + 63) / 64), v_rows((V + 63) / 64 * 64), k_stage((size_t)(chunks_d + chunks_r) * kKChunk),
+          v_stage((size_t)v_rows * 128), q(0), k(q + (size_t)(chunks_d + chunks_r) * kQChunk), v(k + 2 * k_stage), p(v + 2 * v_stage),
+          bars(p + 4 * (size_t)kPBytes), total(bars + 256 + 4 * kRows * sizeof(float)) {}
+};
+
+struct Bars {
+    uint64_t q_full, q_ready, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], o_done[2];
+    uint32_t tmem;
+    int abort;
+};
+
+__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+          "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+        : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};" ::"r"(r[0]), "r"(r[1]),
+        "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]),
+        "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
+        : "memory");
+    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+}
+
+__global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __grid_constant__ LatentParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t *base = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const Layout lay(p.D, p.R, p.V);
+    Bars *b = reinterpret_cast<Bars *>(base + lay.bars);
+    float *stat = reinterpret_cast<float *>(base + lay.bars + 256);  // [2][128] maxima, [2][128] sums
+    volatile int *abort_flag = &b->abort;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int head = blockIdx.x, row0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kRows;  // later rows first: they have the most keys
+    const int last_row = row0 + kRows < p.m ? row0 + kRows - 1 : p.m - 1;
+    const int n_tiles = (p.pos0 + last_row) / kTile + 1;
+    if (tid == 0) {
+        mbar_init(&b->q_full, 1);
+        mbar_init(&b->q_ready, 2 * kGroup);
+        for (int s = 0; s < 2; s++) {
+            mbar_init(&b->k_full[s], 1);
+            mbar_init(&b->k_empty[s], 1);
+            mbar_init(&b->v_full[s], 1);
+            mbar_init(&b->v_empty[s], 1);
+            mbar_init(&b->s_full[s], 1);
+            mbar_init(&b->p_full[s], kGroup);
+            mbar_init(&b->o_done[s], 1);
+        }
+        b->abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&b->tmem)), "r"(512u) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = b->tmem;
+    const uint32_t tm_s[2] = {tmem, tmem + kTile}, tm_o[2] = {tmem + 2 * kTile, tmem + 2 * kTile + (uint32_t)p.V};
+    pdl_enter();
+
+    if (warp == 0) {
+        if (lane == 0) {
+            const int x_q = head * (p.D + p.R), x_k = head * p.D;
+            {
+                mbar_arrive_expect_tx(&b->q_full, (uint32_t)((lay.chunks_d + lay.chunks_r) * kQChunk));
+                const uint32_t at = smem_u32(base + lay.q), bar = smem_u32(&b->q_full);
+                for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kQChunk, p.q_map, x_q + 64 * c, row0, bar);
+                for (int c = 0; c < lay.chunks_r; c++)
+                    tma_load_2d(at + (lay.chunks_d + c) * kQChunk, p.q_map, x_q + p.D + 64 * c, row0, bar);
+            }
+            int j = 0;
+            for (; j < n_tiles; j++) {
+                const int st = j & 1;
+                const uint32_t free_parity = ((j >> 1) & 1u) ^ 1u;
+                if (!mbar_wait(&b->k_empty[st], free_parity, abort_flag, p.status, 31, p.wait_ns)) break;
+                mbar_arrive_expect_tx(&b->k_full[st], (uint32_t)lay.k_stage);
+                uint32_t at = smem_u32(base + lay.k + st * lay.k_stage), bar = smem_u32(&b->k_full[st]);
+                for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kKChunk, p.k_map, x_k + 64 * c, j * kTile, bar);
+                for (int c = 0; c < lay.chunks_r; c++)
+                    tma_load_2d(at + (lay.chunks_d + c) * kKChunk, p.rot_map, 64 * c, p.slot0 * p.max_seq + j * kTile, bar);
+                if (!mbar_wait(&b->v_empty[st], free_parity, abort_flag, p.status, 32, p.wait_ns)) break;
+                mbar_arrive_expect_tx(&b->v_full[st], (uint32_t)lay.v_stage);
+                at = smem_u32(base + lay.v + st * lay.v_stage);
+                bar = smem_u32(&b->v_full[st]);
+                for (int r = 0; r < lay.v_rows; r += 64) tma_load_2d(at + r * 128, p.v_map, j * kTile, head * p.V + r, bar);
+            }
+            if (*abort_flag) {  // no copy may be in flight when the CTA ends
+                mbar_wait(&b->q_full, 0, abort_flag, p.status, 33, p.wait_ns);
+                for (int i = j - 2 > 0 ? j - 2 : 0; i <= j && i < n_tiles; i++) {
+                    mbar_wait(&b->k_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
+                    if (i < j) mbar_wait(&b->v_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
+                }
+            }
+        }
+        __syncwarp();
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc_s = tlc_gemm::idesc_for(kTile) | kIdesc, idesc_o = tlc_gemm::idesc_for(p.V) | kIdesc;
+            auto scores = [&](int j) {
+                const int st = j & 1;
+                if (!mbar_wait(&b->k_full[st], (j >> 1) & 1u, abort_flag, p.status, 34, p.wait_ns)) return false;
+                tc_fence_after();
+                const uint32_t qa = smem_u32(base + lay.q), ka = smem_u32(base + lay.k + st * lay.k_stage);
+                for (int kk = 0; kk < p.D / 16; kk++)
+                    umma_f16(tm_s[st], make_desc(qa + (kk >> 2) * kQChunk + (kk & 3) * 32), make_desc(ka + (kk >> 2) * kKChunk + (kk & 3) * 32),
+                             idesc_s, kk > 0 ? 1u : 0u);
+                for (int kk = 0; kk < p.R / 16; kk++)
+                    umma_f16(tm_s[st], make_desc(qa + (lay.chunks_d + (kk >> 2)) * kQChunk + (kk & 3) * 32),
+                             make_desc(ka + (lay.chunks_d + (kk >> 2)) * kKChunk + (kk & 3) * 32), idesc_s, 1u);
+                umma_commit(&b->k_empty[st]);
+                umma_commit(&b->s_full[st]);
+                return true;
+            };
+            bool ok = mbar_wait(&b->q_ready, 0, abort_flag, p.status, 35, p.wait_ns);
+            tc_fence_after();
+            ok = ok && scores(0);
+            for (int j = 0; ok && j < n_tiles; j++) {
+                // the scores' buffer is free: its group has handed in the weights of tile j - 1
+                if (j + 1 < n_tiles && !scores(j + 1)) break;
+                const int g = j & 1;
+                if (!mbar_wait(&b->p_full[g], (j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
+                if (!mbar_wait(&b->v_full[g], (j >> 1) & 1u, abort_flag, p.status, 37, p.wait_ns)) break;
+                tc_fence_after();
+                const uint32_t va = smem_u32(base + lay.v + g * lay.v_stage);
+#pragma unroll
+                for (int part = 0; part < 2; part++) {
+                    const uint32_t pa = smem_u32(base + lay.p + (size_t)(2 * g + part) * kPBytes);
+#pragma unroll
+                    for (int kk = 0; kk < kTile / 16; kk++)
+                        umma_f16(tm_o[g], make_desc(pa + kk * 32), make_desc(va + kk * 32), idesc_o, j > 1 || part > 0 || kk > 0 ? 1u : 0u);
+                }
+                umma_commit(&b->v_empty[g]);
+                umma_commit(&b->o_done[g]);
+            }
+        }
+        __syncwarp();
+    } else {
+        const int g = (warp - 2) >> 2, wq = warp & 3, r = 32 * wq + lane;  // tensor-memory lanes this warp may touch: 32 wq ..
+        const uint32_t lanes = (uint32_t)(32 * wq) << 16;
+        const int pos = p.pos0 + row0 + r, warp_first = p.pos0 + row0 + 32 * wq;
+        // rotate the queries: the groups share a row's pairs
+        mbar_wait(&b->q_full, 0, abort_flag, p.status, 38, p.wait_ns);
+        for (int i = 4 * g; i < p.R / 2; i += 8) {  // four pairs: one 16-byte piece
+            const int e = 2 * i, c = e >> 6, piece = (e & 63) >> 3;
+            uint4 *at = reinterpret_cast<uint4 *>(base + lay.q + (size_t)(lay.chunks_d + c) * kQChunk + r * 128 + ((piece ^ (r & 7)) << 4));
+            float f[8];
+            unpack(*at, f);
+            uint32_t o[4];
+#pragma unroll
+            for (int t = 0; t < 4; t++) {
+                float sn, cs;
+                sincosf((float)pos * __ldg(p.freq + i + t), &sn, &cs);
+                o[t] = pack_bf16(f[2 * t] * cs - f[2 * t + 1] * sn, f[2 * t + 1] * cs + f[2 * t] * sn);
+            }
+            *at = make_uint4(o[0], o[1], o[2], o[3]);
+        }
+        fence_async_proxy();
+        mbar_arrive(&b->q_ready);
+
+        const float scale2 = p.scale * kLog2e;
+        float m = -INFINITY, l = 0.f;
+        uint8_t *ph = base + lay.p + (size_t)(2 * g) * kPBytes + r * 128, *pl = ph + kPBytes;
+        int it = 0;
+        for (int j = g; j < n_tiles; j += 2, it++) {
+            mbar_wait(&b->s_full[g], it & 1u, abort_flag, p.status, 39, p.wait_ns);
+            tc_fence_after();
+            uint32_t s[2][32];
+            tmem_ld32(tm_s[g] + lanes, s[0]);
+            tmem_ld32(tm_s[g] + lanes + 32, s[1]);
+            const int j0 = j * kTile;
+            float mx0 = -INFINITY, mx1 = -INFINITY;
+            if (j0 + kTile - 1 > warp_first) {  // some row of the warp does not see every key
+#pragma unroll
+                for (int e = 0; e < 32; e++) {
+                    if (j0 + e > pos) s[0][e] = 0xff800000u;
+                    if (j0 + 32 + e > pos) s[1][e] = 0xff800000u;
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 32; e++) {
+                mx0 = fmaxf(mx0, __uint_as_float(s[0][e]));
+                mx1 = fmaxf(mx1, __uint_as_float(s[1][e]));
+            }
+            // the smallest score stands for the maximum when the scale is negative: no assumption on its sign
+            float top = fmaxf(mx0, mx1) * scale2;
+            if (scale2 <= 0.f) {
+                top = -INFINITY;
+#pragma unroll
+                for (int e = 0; e < 32; e++) {
+                    if (j0 + e <= pos) top = fmaxf(top, __uint_as_float(s[0][e]) * scale2);
+                    if (j0 + 32 + e <= pos) top = fmaxf(top, __uint_as_float(s[1][e]) * scale2);
+                }
+            }
+            if (it > 0) mbar_wait(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
+            if (it == 0) {
+                m = top;
+            } else if (__any_sync(0xffffffffu, top > m + 8.f)) {
+                const float m_new = fmaxf(m, top), f = m_new == -INFINITY ? 1.f : exp2f(m - m_new);
+                tc_fence_after();
+                for (int c = 0; c < p.V; c += 16) {
+                    uint32_t o[16];
+                    tmem_ld16(tm_o[g] + lanes + c, o);
+#pragma unroll
+                    for (int e = 0; e < 16; e++) o[e] = __float_as_uint(__uint_as_float(o[e]) * f);
+                    tmem_st16(tm_o[g] + lanes + c, o);
+                }
+                l *= f;
+                m = m_new;
+            }
+            const float from = m == -INFINITY ? 0.f : m;
+            float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+            for (int c = 0; c < 8; c++) {  // eight keys: one 16-byte piece of each part
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int t = 0; t < 4; t++) {
+                    const int e = 8 * (c & 3) + 2 * t;
+                    const uint32_t *v = s[c >> 2];
+                    float a = exp2f(fmaf(__uint_as_float(v[e]), scale2, -from)), d = exp2f(fmaf(__uint_as_float(v[e + 1]), scale2, -from));
+                    if (scale2 <= 0.f) {
+                        a = j0 + 8 * c + 2 * t <= pos ? a : 0.f;
+                        d = j0 + 8 * c + 2 * t + 1 <= pos ? d : 0.f;
+                    }
+                    sum0 += a;
+                    sum1 += d;
+                    split_pair(a, d, hi[t], lo[t]);
+                }
+                *reinterpret_cast<uint4 *>(ph + ((c ^ (r & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                *reinterpret_cast<uint4 *>(pl + ((c ^ (r & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+            l += sum0 + sum1;
+            fence_async_proxy();
+            tc_fence_before();
+            mbar_arrive(&b->p_full[g]);
+        }
+        if (it > 0) mbar_wait(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 41, p.wait_ns);
+        stat[g * kRows + r] = m;
+        stat[(2 + g) * kRows + r] = l;
+        tc_fence_before();
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        tc_fence_after();
+        const float sink = to_f32(static_cast<const bf16 *>(p.sink)[head]) * kLog2e;
+        const float m0 = stat[r], m1 = stat[kRows + r], top = fmaxf(fmaxf(m0, m1), sink);
+        const float e0 = exp2f(m0 - top), e1 = exp2f(m1 - top);
+        const float inv = 1.f / (stat[2 * kRows + r] * e0 + stat[3 * kRows + r] * e1 + exp2f(sink - top));
+        const float f0 = e0 * inv, f1 = e1 * inv;
+        const bool two = n_tiles > 1;  // else the second accumulator was never written
+        bf16 *out = static_cast<bf16 *>(p.out) + (size_t)(row0 + r) * p.ldo + (size_t)head * p.V;
+        const bool store = row0 + r < p.m && !*abort_flag;
+        for (int c = 16 * g; c < p.V; c += 32) {  // the groups take 16 columns in turn
+            uint32_t a[16], d[16];
+            tmem_ld16(tm_o[0] + lanes + c, a);
+            tmem_ld16(tm_o[1] + lanes + c, d);
+            uint32_t o[8];
+#pragma unroll
+            for (int t = 0; t < 8; t++) {
+                float u = __uint_as_float(a[2 * t]) * f0, v = __uint_as_float(a[2 * t + 1]) * f0;
+                if (two) {
+                    u += __uint_as_float(d[2 * t]) * f1;
+                    v += __uint_as_float(d[2 * t + 1]) * f1;
+                }
+                o[t] = pack_bf16(u, v);
+            }
+            if (store) {
+                *reinterpret_cast<uint4 *>(out + c) = make_uint4(o[0], o[1], o[2], o[3]);
+                *reinterpret_cast<uint4 *>(out + c + 8) = make_uint4(o[4], o[5], o[6], o[7]);
+            }
+        }
+        tc_fence_before();
+    }
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+    }
+}
+
+}  // namespace
+
+bool latent_prefill_fits(int D, int R, int V) {
+    static_assert(sizeof(Bars) <= 256, "the barriers have 256 bytes");
+    return D % 16 == 0 && R % 16 == 0 && V % 16 == 0 && D > 0 && V > 0 && 2 * kTile + 2 * V <= 512 &&
+           Layout(D, R, V).total + 1024 <= 227 * 1024;
+}
+
+int32_t launch_latent_prefill(tlc_ctx *ctx, const LatentParams &p) {
+    TLC_REQUIRE(latent_prefill_fits(p.D, p.R, p.V), TLC_ERR_INVALID_OPERATION, "latent attention: heads of %d + %d and %d values", p.D,
+                p.R, p.V);
+    static bool done[64] = {};
+    if (!done[ctx->device & 63]) {
+        TLC_CUDA(cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+        done[ctx->device & 63] = true;
+    }
+    cudaError_t le = tlc_launch_pdl(ctx, latent_prefill_kernel, dim3((unsigned)p.H, (unsigned)((p.m + kRows - 1) / kRows)), dim3(kThreadsP),
+                                    Layout(p.D, p.R, p.V).total + 1024, p);
+    if (le != cudaSuccess) {
+        cudaGetLastError();
+        return tlc_fail(TLC_ERR_CUDA, "latent attention launch failed: %s", cudaGetErrorString(le));
+    }
+    TLC_CHECK_LAUNCH(ctx);
+    return TLC_OK;
 }
 
 }  // namespace tlc_dense
