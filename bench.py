@@ -847,28 +847,48 @@ def toposun_sizes() -> dict:
             "experts": experts(2048, 16, 4, 128, 64, 8, 1024, 2048, 8)}
 
 
-def run_toposun(args) -> None:
-    """--workload toposun --size small|wide|experts: Toposun at the sizes of a real model's layers (random
-    weights, bf16), prompt of 2048 tokens and greedy decode of one sequence behind it, beside the LLaMA
-    runner at the same widths with Q8_0 weights.  Prefill: whole calls from the ids on the host to the
-    sampled token back; decode: graph replays between two CUDA events.  Every step reads more weight
-    bytes than the L2 holds."""
+def suselorn_sizes() -> dict:
+    """name -> (Suselorn, four residual streams; Toposun with the same width, query heads, values and feed-forward, every
+    key visible)."""
+    from tensorlogic_b200.decoder import DecoderArch, LatentLayerArch, LayerArch
+
+    def pair(width, heads, q_rank, ff, n):
+        l = LatentLayerArch(heads, 128, 64, 128, q_rank, 512, 10000.0, 192 ** -0.5, "silu_glu", ff)
+        t = LayerArch(heads, heads // 4, 128, 1 << 20, 0, 128, 10000.0, 128 ** -0.5, "clamped_glu", ff, 7.0)
+        return (DecoderArch(width, 32000, 1e-6, [l] * n, streams=4, logit_softcap=30.0), DecoderArch(width, 32000, 1e-5, [t] * n))
+    return {"small": pair(2048, 16, 768, 5632, 22), "wide": pair(4096, 32, 1536, 11008, 8)}
+
+
+def run_decoder(args) -> None:
+    """--workload toposun | suselorn --size ...: a config-driven decoder at the sizes of a real model's layers
+    (random weights, bf16), prompt of 2048 tokens and greedy decode of one sequence behind it, beside the closest
+    other runner: Toposun beside the LLaMA runner at the same widths with Q8_0 weights, Suselorn beside
+    Toposun.  Prefill: whole calls from the ids on the host to the sampled token back; decode: graph replays
+    between two CUDA events.  Every step reads more weight bytes than the L2 holds."""
     import torch
     from tensorlogic_b200 import synth
     from tensorlogic_b200.api import Device
     from tensorlogic_b200.decoder import Decoder, synthetic_decoder
     from tensorlogic_b200.model import Llama, synthetic_model
     tokens, K, W = 2048, args.steps, max(args.warmup, 3)
-    arch, twin = toposun_sizes()[args.size]
-    if args.window:
+    name = args.workload
+    sizes = toposun_sizes() if name == "toposun" else suselorn_sizes()
+    if args.size not in sizes:
+        raise SystemExit(f"--workload {name} has the sizes {', '.join(sizes)}")
+    arch, twin = sizes[args.size]
+    if args.window and name == "toposun":
         arch.layers = [dataclasses.replace(l, window=args.window) for l in arch.layers]
     if args.layers:
-        arch.layers, twin.n_layers = arch.layers[:args.layers], min(args.layers, twin.n_layers)
+        arch.layers = arch.layers[:args.layers]
+        if name == "toposun":
+            twin.n_layers = min(args.layers, twin.n_layers)
+        else:
+            twin.layers = twin.layers[:args.layers]
     KP = max(3, min(K, 20))
     dev = Device(0)
     peaks = load_peaks()
     stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
-    ids = synth.token_ids(SEED, "toposun.prompt", tokens, arch.vocab)
+    ids = synth.token_ids(SEED, f"{name}.prompt", tokens, arch.vocab)
     max_seq = tokens + W + K + 16
 
     def barrier():
@@ -898,12 +918,15 @@ def run_toposun(args) -> None:
                 "launches_per_step": launches / K, "prefill_tokens_per_s": tokens / pre * 1e3, "prefill_ms": pre,
                 "prefill_tflops": flops / pre / 1e9, "prefill_frac": flops / pre / 1e9 / peaks["bf16_tflops_sustained"]}
 
-    runner = Decoder(dev, synthetic_decoder(dev, arch, SEED), arch, max_seq=max_seq, max_prefill=tokens)
-    weights = sum(arch.layer_weight_bytes(l) for l in arch.layers)
-    kv = sum(2 * 2 * l.kv_heads * l.dim * min(tokens, l.window + l.keep_first) for l in arch.layers)
+    def measure_decoder(arch, clocks=None):
+        runner = Decoder(dev, synthetic_decoder(dev, arch, SEED), arch, max_seq=max_seq, max_prefill=tokens)
+        weights = sum(arch.layer_weight_bytes(l) for l in arch.layers)
+        kv = sum(2 * (l.kv_rank + l.rot_dim) * tokens if arch.streams else
+                 2 * 2 * l.kv_heads * l.dim * min(tokens, l.window + l.keep_first) for l in arch.layers)
+        return runner, measure(runner, weights, arch.vocab * arch.width * 2, kv, weights // 2, clocks)
     launches0 = dev.launch_count
     with ClockSampler(0) as clocks:
-        ours = measure(runner, weights, arch.vocab * arch.width * 2, kv, weights // 2, clocks)
+        runner, ours = measure_decoder(arch, clocks)
     launches = dev.launch_count - launches0
     clock_line = clocks.summary()
     runner.prefill(ids, return_logits=False)
@@ -916,35 +939,40 @@ def run_toposun(args) -> None:
     closest = None
     if not args.no_closest:
         del runner
+    if not args.no_closest and name == "suselorn":
+        runner, closest = measure_decoder(twin)
+        closest["model"] = "toposun, same width, query heads, values and feed-forward; every key visible"
+    elif not args.no_closest:
         llm = Llama(dev, synthetic_model(dev, twin, SEED, qtype=8, device_embeddings=True), twin, max_seq=max_seq, max_prefill=tokens)
         params = sum(r * c for n, (r, c) in twin.tensor_shapes().items() if n.startswith("blk.") and not n.endswith("norm.weight"))
         closest = measure(llm, params // 32 * 34, twin.vocab * twin.d_model // 32 * 34,
                           twin.n_layers * 2 * 2 * twin.n_kv_heads * twin.head_dim * tokens, params)
         closest["model"] = "llama q8_0, same widths, heads and active feed-forward; full causal attention"
     print(json.dumps({
-        "metric": "toposun_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "metric": f"{name}_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
         "steps": K, "warmup": W, "ms_per_step": ours["decode_ms"], "higher_is_better": True, "scaling": "weak",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"model": f"toposun-{args.size}", "layers": len(arch.layers), "width": arch.width, "global_batch": 1,
-                   "seq_len": tokens, "window": arch.layers[0].window, "parallelism": "single",
+        "config": {"model": f"{name}-{args.size}", "layers": len(arch.layers), "width": arch.width, "global_batch": 1, "seq_len": tokens,
+                   **({"streams": arch.streams} if arch.streams else {"window": arch.layers[0].window}), "parallelism": "single",
                    "l2": "the weights of a step exceed the 126 MB L2", "seed": SEED},
         "e2e": {"value": e2e, "unit": "tokens/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4},
-        "gpu_launches": int(launches), "clocks": clock_line, "toposun": ours, "closest": closest,
+        "gpu_launches": int(launches), "clocks": clock_line, name: ours, "closest": closest,
         "peaks": peaks}), flush=True)
 
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "decode70b", "toposun"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "decode70b", "toposun", "suselorn"],
                     help="decode: the headline workload (default); prefill: Llama-2-7B-shape 2048-token prefill; "
                          "toposun: the Toposun decoder (--size) beside the LLaMA runner at equal widths; "
+                         "suselorn: the Suselorn decoder (--size) beside Toposun at equal widths; "
                          "decode70b: the Llama-2-70B-shape decode of the N > 1 runs on ONE GPU (the TP1 point)")
     ap.add_argument("--kernel", default=None, choices=["linear", "allreduce"],
                     help="micro-benchmark one kernel instead of the decode workload (see run_kernel)")
-    ap.add_argument("--size", default="small", choices=["small", "wide", "experts"], help="of --workload toposun")
-    ap.add_argument("--layers", type=int, default=0, help="--workload toposun: only the first so many layers (for profiles)")
+    ap.add_argument("--size", default="small", choices=["small", "wide", "experts"], help="of --workload toposun | suselorn (experts: toposun only)")
+    ap.add_argument("--layers", type=int, default=0, help="--workload toposun | suselorn: only the first so many layers (for profiles)")
     ap.add_argument("--window", type=int, default=0, help="--workload toposun: another window than 1024")
-    ap.add_argument("--no-closest", action="store_true", help="--workload toposun: leave the LLaMA runner out")
+    ap.add_argument("--no-closest", action="store_true", help="--workload toposun | suselorn: leave the other runner out")
     ap.add_argument("--qtype", default="q4_0", choices=["q4_0", "q8_0"])
     ap.add_argument("--n", type=int, default=28672)
     ap.add_argument("--k", type=int, default=8192)
@@ -970,10 +998,10 @@ def main() -> None:
     if args.kernel == "linear":
         run_kernel(args)
         return
-    if args.workload == "toposun":
+    if args.workload in ("toposun", "suselorn"):
         if world > 1:
-            raise SystemExit("--workload toposun runs on one GPU")
-        run_toposun(args)
+            raise SystemExit(f"--workload {args.workload} runs on one GPU")
+        run_decoder(args)
         return
     if world > 1:
         dist_setup(args.gpus)
