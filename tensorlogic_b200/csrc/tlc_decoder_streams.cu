@@ -52,7 +52,7 @@ int32_t host_values(tlc_decoder *D, const tlc_qtensor *t, std::vector<float> *ou
 }
 
 bool expands(const tlc_decoder *D, const tlc_decoder_layer &c) {
-    return D->cfg.dtype == TLC_TYPE_BF16 && latent_prefill_fits(c.dim, c.rot_dims, c.vdim);
+    return D->cfg.dtype == TLC_TYPE_BF16 && latent_prefill_fits(c.dim, c.rot_dims, c.vdim, c.scale);
 }
 
 // The streams' update behind sublayer q of `L`, with the next sublayer's norm; h: its input or null.

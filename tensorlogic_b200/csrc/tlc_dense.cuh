@@ -124,23 +124,29 @@ struct StreamsOut {
 };
 #ifdef __CUDACC__
 __device__ __forceinline__ float tanh_norm(float u, float alpha, float w, float b) { return tanhf(alpha * u) * w + b; }
-// One column: `x` holds the old streams and receives the new ones; returns the next sublayer's u.
+// One column: `x` holds the old streams and receives the new ones; returns the next sublayer's u.  MAXS up to 4
+// is the number of streams, larger only a bound.
+template <int MAXS>
+__device__ __forceinline__ int stream_count(const StreamsOut &o) {
+    return MAXS <= 4 ? MAXS : o.n;
+}
 template <int MAXS>
 __device__ __forceinline__ float update_streams(const StreamsOut &o, float y, float (&x)[MAXS]) {
+    const int n = stream_count<MAXS>(o);
     float nw[MAXS], u = 0.f;
 #pragma unroll
     for (int t = 0; t < MAXS; t++) {
-        if (t >= o.n) break;
+        if (t >= n) continue;
         float v = o.out[t] * y;
 #pragma unroll
         for (int s = 0; s < MAXS; s++)
-            if (s < o.n) v = fmaf(o.mix[s][t], x[s], v);
+            if (s < n) v = fmaf(o.mix[s][t], x[s], v);
         nw[t] = v;
         u = fmaf(o.in[t], v, u);
     }
 #pragma unroll
     for (int t = 0; t < MAXS; t++)
-        if (t < o.n) x[t] = nw[t];
+        if (t < n) x[t] = nw[t];
     return u;
 }
 // The same with loads and stores, for column n of row `row` and the finished product `acc`.
@@ -419,6 +425,6 @@ int32_t launch_latent_absorbed(tlc_ctx *ctx, const LatentParams &p);
 int latent_splits(const tlc_ctx *ctx, const LatentParams &p);  // stretches for p.m rows of p.H heads
 // Expanded: attention of consecutive rows over k_all, v_all and the cache's rotated parts (bf16).
 int32_t launch_latent_prefill(tlc_ctx *ctx, const LatentParams &p);
-bool latent_prefill_fits(int D, int R, int V);
+bool latent_prefill_fits(int D, int R, int V, float scale);
 
 }  // namespace tlc_dense

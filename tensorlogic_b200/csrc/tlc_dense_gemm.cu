@@ -228,7 +228,7 @@ __device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsO
                 const int r = 8 * (i0 + i) + (lane >> 2);
 #pragma unroll
                 for (int s = 0; s < MAXS; s++)
-                    if (s < st.n && r < rows)
+                    if (s < stream_count<MAXS>(st) && r < rows)
                         x[i][s] = __ldcg(reinterpret_cast<const float4 *>(st.x + s * st.plane + (int64_t)(row0 + r) * g.n + n));
             }
 #pragma unroll
@@ -255,7 +255,7 @@ __device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsO
                 }
 #pragma unroll
                 for (int s = 0; s < MAXS; s++)
-                    if (s < st.n) *reinterpret_cast<float4 *>(st.x + s * st.plane + (int64_t)(row0 + r) * g.n + n) = x[i][s];
+                    if (s < stream_count<MAXS>(st)) *reinterpret_cast<float4 *>(st.x + s * st.plane + (int64_t)(row0 + r) * g.n + n) = x[i][s];
                 if (st.h) {
                     const __nv_bfloat162 lo = __floats2bfloat162_rn(h[0], h[1]), hi = __floats2bfloat162_rn(h[2], h[3]);
                     *reinterpret_cast<uint2 *>(static_cast<bf16 *>(st.h) + (int64_t)(row0 + r) * st.ldh + n) =
@@ -266,7 +266,7 @@ __device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsO
     }
 }
 
-// MAXS > 0: the form whose groups end in EPI_STREAMS, for up to MAXS streams.
+// MAXS > 0: the form whose group ends in EPI_STREAMS, for MAXS streams (8: for up to so many).
 template <int MAXS>
 __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -369,6 +369,13 @@ __global__ void __launch_bounds__(kThreadsD, 1) dense_gemm_kernel(const __grid_c
             const Tile tl = tile_at<128, 256>(p, start, first_row, t, slot);
             const GemmGroup &g = p.g[tl.group];
             const int a = it & 1;
+            if constexpr (MAXS > 0) {  // the old streams on their way to the L2 while the tile's products run
+                if ((g.n & 3) == 0)
+                    for (int i = tid - 64; i < tl.rows * p.st.n; i += 32 * kEpilogueWarps) {
+                        const int s = i / tl.rows, n = g.n - tl.n0 < 256 ? g.n - tl.n0 : 256;
+                        prefetch_l2(p.st.x + s * p.st.plane + (int64_t)(tl.row0 + i - s * tl.rows) * g.n + tl.n0, (uint32_t)n * 4);
+                    }
+            }
             const bool done = mbar_wait(&acc_full[a], (it >> 1) & 1u, abort_flag, p.status, 24, p.wait_ns);
             tc_fence_after();
             const int row = 32 * wq + lane;
@@ -559,7 +566,13 @@ int32_t launch_gemm<bf16>(tlc_ctx *ctx, GemmParams &p) {
     long tiles = tile_bound(p, 128, 256, 128, family);
     if (tiles > ctx->sm_count) tiles = ctx->sm_count;
     if (p.st.n == 0) return launch_tensor<0>(ctx, p, tiles);
-    return p.st.n <= 4 ? launch_tensor<4>(ctx, p, tiles) : launch_tensor<kMaxStreams>(ctx, p, tiles);
+    switch (p.st.n) {
+        case 1: return launch_tensor<1>(ctx, p, tiles);
+        case 2: return launch_tensor<2>(ctx, p, tiles);
+        case 3: return launch_tensor<3>(ctx, p, tiles);
+        case 4: return launch_tensor<4>(ctx, p, tiles);
+        default: return launch_tensor<kMaxStreams>(ctx, p, tiles);
+    }
 }
 
 template <>

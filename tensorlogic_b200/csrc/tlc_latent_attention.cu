@@ -14,14 +14,17 @@
 //
 // Scores, statistics and weights are f32; a weight enters the tensor-core product as the sum of two bf16
 // numbers (high and low part).
+#include <algorithm>
+
 #include "tlc_dense.cuh"
 #include "tlc_mma.cuh"
+#include "tlc_stream.cuh"
 
 namespace tlc_dense {
 
 namespace {
 
-constexpr int kQueryThreads = 256, kScanThreads = 256, kScanWarps = kScanThreads / 32, kValueThreads = 256;
+constexpr int kQueryThreads = 512, kScanThreads = 256, kScanWarps = kScanThreads / 32, kValueThreads = 512;
 constexpr int kKeys = 64;       // keys per tile
 constexpr int kTileHeads = 16;
 constexpr int kPPitch = kKeys + 8;
@@ -36,25 +39,48 @@ __device__ __forceinline__ float2 rotate_pair(float u, float v, int pos, float f
     return make_float2(u * cs - v * sn, v * cs + u * sn);
 }
 
-// Row r's latent, normalized, and its rotated key part into the cache.  All threads of the block.
+// 1 / root mean square of n values of a row padded to whole pieces, by one warp.
 template <typename T>
-__device__ void append_latent(const LatentParams &p, int r, float *red) {
-    const T *z = static_cast<const T *>(p.ckv_raw) + (size_t)r * p.ldckv, *w = static_cast<const T *>(p.dkv_norm);
-    const int tid = threadIdx.x, n = blockDim.x;
+__device__ __forceinline__ float warp_rms(const T *z, int n, float eps, int lane) {
+    constexpr int N = Vec<T>::N;
     float s = 0.f;
-    for (int i = tid; i < p.KR; i += n) {
-        const float v = to_f32(z[i]);
-        s += v * v;
+#pragma unroll 4
+    for (int c = lane; N * c < n; c += 32) {
+        float f[N];
+        unpack(__ldcg(reinterpret_cast<const uint4 *>(z) + c), f);
+#pragma unroll
+        for (int e = 0; e < N; e++) s += N * c + e < n ? f[e] * f[e] : 0.f;
     }
-    const float rstd = 1.0f / sqrtf(block_sum(s, red) / (float)p.KR + p.eps);
+    return 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
+}
+// out = z * rstd * w in whole pieces; w is padded with zeros.
+template <typename T>
+__device__ __forceinline__ void warp_scale(const T *z, const T *w, T *out, int n, float rstd, int lane) {
+    constexpr int N = Vec<T>::N;
+#pragma unroll 4
+    for (int c = lane; N * c < n; c += 32) {
+        float f[N], g[N];
+        unpack(__ldcg(reinterpret_cast<const uint4 *>(z) + c), f);
+        unpack(load_nc(w + N * c), g);
+        union { uint4 v; T t[N]; } o;
+#pragma unroll
+        for (int e = 0; e < N; e++) o.t[e] = from_f32<T>(N * c + e < n ? f[e] * rstd * g[e] : 0.f);
+        reinterpret_cast<uint4 *>(out)[c] = o.v;
+    }
+}
+
+// Row r's latent, normalized, and its rotated key part into the cache.  One warp.
+template <typename T>
+__device__ void append_latent(const LatentParams &p, int r, int lane) {
+    const T *z = static_cast<const T *>(p.ckv_raw) + (size_t)r * p.ldckv;
     const int pos = p.pos[r];
     if (pos < 0 || pos >= p.max_seq) {  // a cache row that does not exist: nothing is written, the host hears about it
-        if (tid == 0 && atomicCAS(&p.status->code, 0, TLC_DEV_INDEX) == 0) p.status->where = 411;
+        if (lane == 0 && atomicCAS(&p.status->code, 0, TLC_DEV_INDEX) == 0) p.status->where = 411;
         return;
     }
     T *row = static_cast<T *>(p.cache) + ((size_t)p.slot[r] * p.max_seq + pos) * p.row;
-    for (int i = tid; i < p.kp; i += n) row[i] = from_f32<T>(i < p.KR ? to_f32(z[i]) * rstd * to_f32(w[i]) : 0.f);
-    for (int i = tid; i < (p.row - p.kp) / 2; i += n) {
+    warp_scale(z, static_cast<const T *>(p.dkv_norm), row, p.KR, warp_rms(z, p.KR, p.eps, lane), lane);
+    for (int i = lane; i < (p.row - p.kp) / 2; i += 32) {
         float2 v = make_float2(0.f, 0.f);
         if (2 * i < p.R) v = rotate_pair(to_f32(z[p.KR + 2 * i]), to_f32(z[p.KR + 2 * i + 1]), pos, p.freq[i]);
         row[p.kp + 2 * i] = from_f32<T>(v.x);
@@ -62,24 +88,18 @@ __device__ void append_latent(const LatentParams &p, int r, float *red) {
     }
 }
 
+// A warp per (row, latent of the queries or of the keys).
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rows_kernel(const __grid_constant__ LatentParams p) {
-    __shared__ float red[33];
     pdl_enter();
-    const int r = blockIdx.x, tid = threadIdx.x;
-    if (blockIdx.y == 1) {
-        append_latent<T>(p, r, red);
-        return;
+    const int w = blockIdx.x * 8 + (threadIdx.x >> 5), r = w >> 1, lane = threadIdx.x & 31;
+    if (r >= p.m) return;
+    if (w & 1) {
+        append_latent<T>(p, r, lane);
+    } else {
+        const T *z = static_cast<const T *>(p.cq_raw) + (size_t)r * p.ldcq;
+        warp_scale(z, static_cast<const T *>(p.dq_norm), static_cast<T *>(p.cq) + (size_t)r * p.ldcq, p.QR, warp_rms(z, p.QR, p.eps, lane), lane);
     }
-    const T *z = static_cast<const T *>(p.cq_raw) + (size_t)r * p.ldcq, *w = static_cast<const T *>(p.dq_norm);
-    T *out = static_cast<T *>(p.cq) + (size_t)r * p.ldcq;
-    float s = 0.f;
-    for (int i = tid; i < p.QR; i += blockDim.x) {
-        const float v = to_f32(z[i]);
-        s += v * v;
-    }
-    const float rstd = 1.0f / sqrtf(block_sum(s, red) / (float)p.QR + p.eps);
-    for (int i = tid; i < p.QR; i += blockDim.x) out[i] = from_f32<T>(to_f32(z[i]) * rstd * to_f32(w[i]));
 }
 
 __device__ __forceinline__ void store_remote_f32(float *at, int rank, float v) {
@@ -90,97 +110,77 @@ __device__ __forceinline__ void store_remote_f32(float *at, int rank, float v) {
 
 // Grid (C, H [+ 1: the append], rows); the C CTAs of a head are a cluster when p.q is null.
 template <typename T>
-__global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const __grid_constant__ LatentParams p) {
-    constexpr int N = Vec<T>::N;
+__global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __grid_constant__ LatentParams p, int split) {
+    constexpr int N = Vec<T>::N, KEPT = 4;
     extern __shared__ __align__(16) float smem[];
-    __shared__ float red[33];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, C = gridDim.x, rank = blockIdx.x, head = blockIdx.y,
               r = blockIdx.z;
     if (head == p.H) {
         pdl_enter();
-        if (rank == 0) append_latent<T>(p, r, red);
+        if (rank == 0 && warp == 0) append_latent<T>(p, r, lane);
         return;
     }
-    const int DR = p.D + p.R, qpieces = (p.QR + N - 1) / N;
-    float *qs = smem;                           // [DR]: the head's query
-    float *cq = qs + ((DR + 3) & ~3);           // [qpieces * N]
-    float *sums = cq + (p.q ? 0 : qpieces * N); // [kQueryThreads][N]
+    const int DR = p.D + p.R, qpieces = (p.QR + N - 1) / N, rows = (DR + C - 1) / C;
+    float *qs = smem;                               // [DR]: the head's query
+    float *cq = qs + ((DR + 3) & ~3);               // [qpieces * N], in the places of put_piece
+    float *sums = cq + (p.q ? 0 : qpieces * N);     // [kQueryThreads][N], before that [rows][split]
     const bool cluster = !p.q && C > 1;
     if (cluster) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // this CTA is running
+    // latent columns of this CTA, in pieces; a thread holds one piece of columns and every `groups`-th d
     const T *uk = static_cast<const T *>(p.uk) + (size_t)head * p.D * p.uk_pitch;
-    const int pieces = (p.KR + N - 1) / N, per = (pieces + C - 1) / C;  // latent columns of this CTA, in pieces
+    const int pieces = (p.KR + N - 1) / N, per = (pieces + C - 1) / C;
     const int p_lo = rank * per < pieces ? rank * per : pieces, p_hi = p_lo + per < pieces ? p_lo + per : pieces;
+    const int np = p_hi - p_lo < kQueryThreads ? p_hi - p_lo : kQueryThreads, groups = np > 0 ? kQueryThreads / np : 0;
+    const int g = np > 0 ? tid / np : 0, c_own = p_lo + tid - g * np;
     const int pos = p.pos[r];  // written at least two kernels ago
+    const int lo = rank * rows, hi = lo + rows < DR ? lo + rows : DR;
+    const T *uq = static_cast<const T *>(p.uq) + (size_t)head * DR * p.uq_pitch;
+    // weights are never written: they can be on their way before the input exists
+    if (!p.q)
+        for (int i = lo + tid; i < hi; i += kQueryThreads) prefetch_l2(uq + (size_t)i * p.uq_pitch, (uint32_t)(qpieces * 16));
+    uint4 kept[KEPT];
+#pragma unroll
+    for (int i = 0; i < KEPT; i++)
+        kept[i] = g < groups && g + i * groups < p.D ? load_weight(reinterpret_cast<const uint4 *>(uk + (size_t)(g + i * groups) * p.uk_pitch) + c_own)
+                                                     : make_uint4(0u, 0u, 0u, 0u);
+    pdl_enter();
     if (p.q) {
-        pdl_enter();
         const T *q = static_cast<const T *>(p.q) + (size_t)r * p.ldq + (size_t)head * DR;
         for (int i = tid; i < DR; i += kQueryThreads) qs[i] = to_f32(q[i]);
         __syncthreads();
     } else {
-        const T *uq = static_cast<const T *>(p.uq) + (size_t)head * DR * p.uq_pitch;
-        const int rows = (DR + C - 1) / C, lo = rank * rows, hi = lo + rows < DR ? lo + rows : DR;
-        // weights are never written: they can be on their way to the L2 before the input exists
-        for (int i = lo + tid; i < hi; i += kQueryThreads) prefetch_l2(uq + (size_t)i * p.uq_pitch, (uint32_t)(qpieces * 16));
-        if (p_hi > p_lo)
-            for (int i = tid; i < p.D; i += kQueryThreads)
-                prefetch_l2(uk + (size_t)i * p.uk_pitch + p_lo * N, (uint32_t)((p_hi - p_lo) * 16));
-        pdl_enter();
         const T *z = static_cast<const T *>(p.cq_raw) + (size_t)r * p.ldcq;
-        float s = 0.f;
-        for (int c = tid; c < qpieces; c += kQueryThreads) {  // rows are padded to whole pieces, with anything
-            float f[N];
-            unpack(__ldcg(reinterpret_cast<const uint4 *>(z) + c), f);
-#pragma unroll
-            for (int e = 0; e < N; e++) s += N * c + e < p.QR ? f[e] * f[e] : 0.f;
-        }
-        const float rstd = 1.0f / sqrtf(block_sum(s, red) / (float)p.QR + p.eps);
+        const float rstd = warp_rms(z, p.QR, p.eps, lane);  // every warp by itself
         for (int c = tid; c < qpieces; c += kQueryThreads) {
             float f[N], w[N];
             unpack(__ldcg(reinterpret_cast<const uint4 *>(z) + c), f);
             unpack(load_nc(static_cast<const T *>(p.dq_norm) + c * N), w);
 #pragma unroll
-            for (int e = 0; e < N; e++) cq[N * c + e] = N * c + e < p.QR ? f[e] * rstd * w[e] : 0.f;
+            for (int e = 0; e < N; e++) f[e] = N * c + e < p.QR ? f[e] * rstd * w[e] : 0.f;
+            put_piece<T>(cq, c, qpieces, f);
         }
         __syncthreads();
+        const int share = (qpieces + split - 1) / split;
+        if (hi > lo)
+            stream_items<T, kQueryThreads / 32>(hi - lo, split, cq, cq + 4 * qpieces, sums, [&](int i, int t) {
+                Item it;
+                it.w = reinterpret_cast<const uint4 *>(uq + (size_t)(lo + i) * p.uq_pitch);
+                share_of(share, qpieces, t, it);
+                it.shift = 0;
+                it.slot = i * split + t;
+                it.scale = 1.f;
+                return it;
+            });
+        __syncthreads();
         if (cluster) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");  // every peer is running
-        constexpr int ROWS = 4;  // rows of a warp in flight
-        for (int i0 = lo + ROWS * warp; i0 < hi; i0 += ROWS * (kQueryThreads / 32)) {
-            float acc[ROWS];
-#pragma unroll
-            for (int j = 0; j < ROWS; j++) acc[j] = 0.f;
-#pragma unroll 2
-            for (int c = lane; c < qpieces; c += 32) {
-                uint4 w[ROWS];
-#pragma unroll
-                for (int j = 0; j < ROWS; j++)
-                    w[j] = i0 + j < hi ? load_nc(uq + (size_t)(i0 + j) * p.uq_pitch + c * N) : make_uint4(0u, 0u, 0u, 0u);
-                float x[N];
-#pragma unroll
-                for (int e = 0; e < N; e += 4) {
-                    const float4 v = *reinterpret_cast<const float4 *>(cq + c * N + e);
-                    x[e] = v.x;
-                    x[e + 1] = v.y;
-                    x[e + 2] = v.z;
-                    x[e + 3] = v.w;
-                }
-#pragma unroll
-                for (int j = 0; j < ROWS; j++) {
-                    float f[N];
-                    unpack(w[j], f);
-#pragma unroll
-                    for (int e = 0; e < N; e++) acc[j] = fmaf(f[e], x[e], acc[j]);
-                }
-            }
-#pragma unroll
-            for (int j = 0; j < ROWS; j++) {
-                acc[j] = warp_sum(acc[j]);
-                if (i0 + j >= hi) continue;
-                if (cluster) {
-                    if (lane < C) store_remote_f32(qs + i0 + j, lane, acc[j]);
-                } else if (lane == 0) {
-                    qs[i0 + j] = acc[j];
-                }
-            }
+        for (int i = tid; i < (hi - lo) * C; i += kQueryThreads) {
+            const int row = i / C, peer = i - row * C;
+            float a = 0.f;
+            for (int t = 0; t < split; t++) a += sums[row * split + t];
+            if (cluster)
+                store_remote_f32(qs + lo + row, peer, a);
+            else
+                qs[lo + row] = a;
         }
         if (cluster) {
             asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
@@ -199,27 +199,33 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const __gri
             out[p.kp + 2 * i + 1] = from_f32<T>(v.y);
         }
     }
-    // q'[column] = sum_d q[d] W_uk[d][column]: a thread holds one piece of columns and every `groups`-th d
-    for (int c0 = p_lo; c0 < p_hi; c0 += kQueryThreads) {
-        const int np = p_hi - c0 < kQueryThreads ? p_hi - c0 : kQueryThreads, groups = kQueryThreads / np;
-        const int g = tid / np, c = c0 + tid - g * np;
+    // q'[column] = sum_d q[d] W_uk[d][column]
+    for (int c0 = p_lo; c0 < p_hi; c0 += np) {
+        const int c = c_own + c0 - p_lo, width = p_hi - c0 < np ? p_hi - c0 : np;  // pieces of this turn
         float acc[N];
 #pragma unroll
         for (int e = 0; e < N; e++) acc[e] = 0.f;
-        if (g < groups)
-#pragma unroll 4
-            for (int d = g; d < p.D; d += groups) {
-                float f[N];
-                unpack(load_nc(uk + (size_t)d * p.uk_pitch + c * N), f);  // rows are padded with zeros
-                const float x = qs[d];
+        auto add = [&](const uint4 &v, int d) {
+            float f[N];
+            unpack(v, f);  // rows are padded with zeros
+            const float x = qs[d];
 #pragma unroll
-                for (int e = 0; e < N; e++) acc[e] = fmaf(f[e], x, acc[e]);
-            }
+            for (int e = 0; e < N; e++) acc[e] = fmaf(f[e], x, acc[e]);
+        };
+        if (g < groups && c < p_hi) {
+            int d = g;
+            if (c0 == p_lo)
+#pragma unroll
+                for (int i = 0; i < KEPT; i++, d += groups)
+                    if (d < p.D) add(kept[i], d);
+#pragma unroll 4
+            for (; d < p.D; d += groups) add(load_weight(reinterpret_cast<const uint4 *>(uk + (size_t)d * p.uk_pitch) + c), d);
+        }
 #pragma unroll
         for (int e = 0; e < N; e += 4)
             *reinterpret_cast<float4 *>(sums + tid * N + e) = make_float4(acc[e], acc[e + 1], acc[e + 2], acc[e + 3]);
         __syncthreads();
-        for (int i = tid; i < np * N; i += kQueryThreads) {
+        for (int i = tid; i < width * N; i += kQueryThreads) {
             float a = 0.f;
             for (int j = 0; j < groups; j++) a += sums[(size_t)j * np * N + i];
             out[c0 * N + i] = from_f32<T>(a);
@@ -475,79 +481,111 @@ __global__ void __launch_bounds__(128) latent_scan_fma_kernel(const __grid_const
 
 // Grid (shares of the head's values, H, rows).
 template <typename T>
-__global__ void __launch_bounds__(kValueThreads) latent_value_kernel(const __grid_constant__ LatentParams p) {
-    constexpr int N = Vec<T>::N;
+__global__ void __launch_bounds__(kValueThreads, 1) latent_value_kernel(const __grid_constant__ LatentParams p) {
+    constexpr int N = Vec<T>::N, WARPS = kValueThreads / 32, KEPT = 2, PARTS = 8;
     extern __shared__ __align__(16) float smem[];
-    float *ol = smem, *f = ol + p.kp;  // the head's weighted latent; factors of the stretches
+    float *ol = smem, *f = ol + p.kp, *sums = f + ((p.nsplit + 3) & ~3);  // the head's weighted latent; factors; [kValueThreads][4]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y, r = blockIdx.z;
     const int per = (p.V + gridDim.x - 1) / gridDim.x, lo = blockIdx.x * per, hi = lo + per < p.V ? lo + per : p.V;
     const T *uv = static_cast<const T *>(p.uv) + (size_t)head * p.V * p.uv_pitch;
     const int pieces = (p.KR + N - 1) / N;
-    for (int i = lo + tid; i < hi; i += kValueThreads) prefetch_l2(uv + (size_t)i * p.uv_pitch, (uint32_t)(pieces * 16));
+    // the first weight rows and pieces of this warp, before the input exists
+    uint4 kept[KEPT][KEPT];
+#pragma unroll
+    for (int k = 0; k < KEPT; k++)
+#pragma unroll
+        for (int u = 0; u < KEPT; u++) {
+            const int i = lo + warp + WARPS * k, c = lane + 32 * u;
+            kept[k][u] = i < hi && c < pieces ? load_weight(reinterpret_cast<const uint4 *>(uv + (size_t)i * p.uv_pitch) + c)
+                                              : make_uint4(0u, 0u, 0u, 0u);
+        }
     const float sink = to_f32(static_cast<const T *>(p.sink)[head]) * kLog2e;
     pdl_enter();
     if (lo >= hi) return;
     const float *stat = p.stat + ((size_t)r * p.nsplit * p.H + head) * 2, *part = p.part + ((size_t)r * p.nsplit * p.H + head) * p.kp;
-    if (warp == 0) {  // factors: exp2(m_s - m) / (sum_s l_s exp2(m_s - m) + exp2(sink - m))
+    const size_t step = (size_t)p.H * p.kp;
+    // a thread adds four columns of every `groups`-th stretch
+    const int quads = p.kp / 4 < kValueThreads ? p.kp / 4 : kValueThreads, groups = kValueThreads / quads, g = tid / quads;
+    float4 v[PARTS];
+#pragma unroll
+    for (int i = 0; i < PARTS; i++)
+        if (g < groups && g + i * groups < p.nsplit)
+            v[i] = __ldcg(reinterpret_cast<const float4 *>(part + (g + i * groups) * step) + (tid - g * quads));
+    {  // factors: exp2(m_s - m) / (sum_s l_s exp2(m_s - m) + exp2(sink - m)); every warp makes them all
         float m = sink;
         for (int s = lane; s < p.nsplit; s += 32) m = fmaxf(m, __ldcg(stat + (size_t)s * p.H * 2));
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
         float l = 0.f;
-        for (int s = lane; s < p.nsplit; s += 32) {
-            const float e = exp2f(__ldcg(stat + (size_t)s * p.H * 2) - m);
-            f[s] = e;
-            l += e * __ldcg(stat + (size_t)s * p.H * 2 + 1);
-        }
+        for (int s = lane; s < p.nsplit; s += 32)
+            l += exp2f(__ldcg(stat + (size_t)s * p.H * 2) - m) * __ldcg(stat + (size_t)s * p.H * 2 + 1);
         l = warp_sum(l) + exp2f(sink - m);
-        for (int s = lane; s < p.nsplit; s += 32) f[s] /= l;
+        if (warp == 0)
+            for (int s = lane; s < p.nsplit; s += 32) f[s] = exp2f(__ldcg(stat + (size_t)s * p.H * 2) - m) / l;
     }
     __syncthreads();
-    for (int c = 4 * tid; c < p.kp; c += 4 * kValueThreads) {
+    for (int q0 = 0; q0 < p.kp / 4; q0 += quads) {
+        const int q = q0 + tid - g * quads;
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-        for (int s = 0; s < p.nsplit; s++) {
-            const float4 v = __ldcg(reinterpret_cast<const float4 *>(part + (size_t)s * p.H * p.kp + c));
+        auto add = [&](const float4 &w, int s) {
             const float e = f[s];
-            a.x = fmaf(e, v.x, a.x);
-            a.y = fmaf(e, v.y, a.y);
-            a.z = fmaf(e, v.z, a.z);
-            a.w = fmaf(e, v.w, a.w);
+            a.x = fmaf(e, w.x, a.x);
+            a.y = fmaf(e, w.y, a.y);
+            a.z = fmaf(e, w.z, a.z);
+            a.w = fmaf(e, w.w, a.w);
+        };
+        if (g < groups && q < p.kp / 4) {
+            int s = g;
+            if (q0 == 0)
+#pragma unroll
+                for (int i = 0; i < PARTS; i++, s += groups)
+                    if (s < p.nsplit) add(v[i], s);
+#pragma unroll 4
+            for (; s < p.nsplit; s += groups) add(__ldcg(reinterpret_cast<const float4 *>(part + s * step) + q), s);
         }
-        *reinterpret_cast<float4 *>(ol + c) = a;
+        *reinterpret_cast<float4 *>(sums + 4 * tid) = a;
+        __syncthreads();
+        for (int i = tid; i < 4 * quads && 4 * q0 + i < p.kp; i += kValueThreads) {
+            float t = 0.f;
+            for (int j = 0; j < groups; j++) t += sums[j * 4 * quads + i];
+            ol[4 * q0 + i] = t;
+        }
+        __syncthreads();
     }
-    __syncthreads();
-    constexpr int ROWS = 4;
     T *out = static_cast<T *>(p.out) + (size_t)r * p.ldo + (size_t)head * p.V;
-    for (int i0 = lo + ROWS * warp; i0 < hi; i0 += ROWS * (kValueThreads / 32)) {
-        float acc[ROWS];
+    auto dot = [&](const uint4 &w, int c) {
+        float x[N], s = 0.f;
+        unpack(w, x);  // rows are padded with zeros
 #pragma unroll
-        for (int j = 0; j < ROWS; j++) acc[j] = 0.f;
-#pragma unroll 2
-        for (int c = lane; c < pieces; c += 32) {
-            float x[N];
-#pragma unroll
-            for (int e = 0; e < N; e += 4) {
-                const float4 v = *reinterpret_cast<const float4 *>(ol + c * N + e);
-                x[e] = v.x;
-                x[e + 1] = v.y;
-                x[e + 2] = v.z;
-                x[e + 3] = v.w;
-            }
-#pragma unroll
-            for (int j = 0; j < ROWS; j++) {
-                if (i0 + j >= hi) continue;
-                float w[N];
-                unpack(load_nc(uv + (size_t)(i0 + j) * p.uv_pitch + c * N), w);  // rows are padded with zeros
-#pragma unroll
-                for (int e = 0; e < N; e++) acc[j] = fmaf(w[e], x[e], acc[j]);
-            }
+        for (int e = 0; e < N; e += 4) {
+            const float4 o = *reinterpret_cast<const float4 *>(ol + c * N + e);
+            s = fmaf(x[e], o.x, s);
+            s = fmaf(x[e + 1], o.y, s);
+            s = fmaf(x[e + 2], o.z, s);
+            s = fmaf(x[e + 3], o.w, s);
         }
+        return s;
+    };
+    auto finish = [&](float acc, int i) {
+        acc = warp_sum(acc);
+        if (lane == 0) out[i] = from_f32<T>(acc);
+    };
 #pragma unroll
-        for (int j = 0; j < ROWS; j++) {
-            acc[j] = warp_sum(acc[j]);
-            if (lane == 0 && i0 + j < hi) out[i0 + j] = from_f32<T>(acc[j]);
-        }
+    for (int k = 0; k < KEPT; k++) {
+        const int i = lo + warp + WARPS * k;
+        if (i >= hi) break;
+        float acc = 0.f;
+#pragma unroll
+        for (int u = 0; u < KEPT; u++)
+            if (lane + 32 * u < pieces) acc += dot(kept[k][u], lane + 32 * u);
+        for (int c = lane + 32 * KEPT; c < pieces; c += 32) acc += dot(load_weight(reinterpret_cast<const uint4 *>(uv + (size_t)i * p.uv_pitch) + c), c);
+        finish(acc, i);
+    }
+    for (int i = lo + warp + WARPS * KEPT; i < hi; i += WARPS) {
+        float acc = 0.f;
+#pragma unroll 4
+        for (int c = lane; c < pieces; c += 32) acc += dot(load_weight(reinterpret_cast<const uint4 *>(uv + (size_t)i * p.uv_pitch) + c), c);
+        finish(acc, i);
     }
 }
 
@@ -590,20 +628,23 @@ int latent_splits(const tlc_ctx *ctx, const LatentParams &p) {
 
 template <typename T>
 int32_t launch_latent_rows(tlc_ctx *ctx, const LatentParams &p) {
-    return launched(ctx, tlc_launch_pdl(ctx, latent_rows_kernel<T>, dim3((unsigned)p.m, 2), dim3(256), 0, p));
+    return launched(ctx, tlc_launch_pdl(ctx, latent_rows_kernel<T>, dim3((unsigned)((2 * p.m + 7) / 8)), dim3(256), 0, p));
 }
 
 template <typename T>
 int32_t launch_latent_query(tlc_ctx *ctx, const LatentParams &p) {
     constexpr int N = Vec<T>::N;
     const int DR = p.D + p.R, qpieces = (p.QR + N - 1) / N;
-    const size_t smem = ((size_t)((DR + 3) & ~3) + (p.q ? 0 : (size_t)qpieces * N) + (size_t)kQueryThreads * N) * sizeof(float);
+    // CTAs per head: enough for the SMs, at most eight (a portable cluster), no more than pieces of the latent
+    int C = 1;
+    while (C < 8 && (long)2 * C * (p.H + 1) * p.m <= ctx->sm_count && 2 * C <= p.kp / N) C *= 2;
+    const int split = (qpieces + 32 * kBatch - 1) / (32 * kBatch);  // stretches a row of W_uq is cut into
+    const size_t area = std::max((size_t)kQueryThreads * N, p.q ? 0 : (size_t)((DR + C - 1) / C) * split);
+    const size_t smem = ((size_t)((DR + 3) & ~3) + (p.q ? 0 : (size_t)qpieces * N) + area) * sizeof(float);
     TLC_REQUIRE(smem <= 200 * 1024, TLC_ERR_INVALID_OPERATION, "latent attention: a query latent of %d and heads of %d + %d do not fit",
                 p.QR, p.D, p.R);
     static bool done[64] = {};
     if (int32_t rc = allow_smem(latent_query_kernel<T>, done, ctx->device, 200 * 1024)) return rc;
-    int C = 1;  // CTAs per head: enough for the SMs, at most eight (a portable cluster), no more than pieces of the latent
-    while (C < 8 && (long)2 * C * p.H * p.m <= ctx->sm_count && 2 * C <= p.kp / N) C *= 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((unsigned)C, (unsigned)(p.q ? p.H : p.H + 1), (unsigned)p.m);
     cfg.blockDim = dim3(kQueryThreads);
@@ -623,7 +664,7 @@ int32_t launch_latent_query(tlc_ctx *ctx, const LatentParams &p) {
     }
     cfg.attrs = attr;
     cfg.numAttrs = n;
-    return launched(ctx, cudaLaunchKernelEx(&cfg, latent_query_kernel<T>, p));
+    return launched(ctx, cudaLaunchKernelEx(&cfg, latent_query_kernel<T>, p, split));
 }
 
 template <typename T>
@@ -642,7 +683,7 @@ int32_t launch_latent_absorbed(tlc_ctx *ctx, const LatentParams &p) {
                                           smem, p));
     }
     if (rc) return rc;
-    const size_t smem = ((size_t)p.kp + p.nsplit) * sizeof(float);
+    const size_t smem = ((size_t)p.kp + ((p.nsplit + 3) & ~3) + 4 * kValueThreads) * sizeof(float);
     TLC_REQUIRE(smem <= 200 * 1024, TLC_ERR_INVALID_OPERATION, "latent attention: a latent of %d values does not fit", p.KR);
     static bool done[64] = {};
     if ((rc = allow_smem(latent_value_kernel<T>, done, ctx->device, 200 * 1024))) return rc;

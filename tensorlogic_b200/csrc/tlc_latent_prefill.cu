@@ -5,10 +5,11 @@
 // rotated part all heads share straight from the cache, values transposed (V rows of 64 keys), so that
 // every operand is K-major; all by TMA with the 128-byte swizzle, two stages.
 //   warp 0       TMA
-//   warp 1       issues the MMAs: S = Q K^T of tile j + 1 before P V of tile j
+//   warp 1       issues the MMAs: S = Q K^T runs up to three tiles ahead of P V (four score buffers; two
+//                when the accumulators leave no more room in the tensor memory)
 //   warps 2-9    two softmax groups of 128 threads, one query row per thread; group g owns the tiles
-//                j = g (mod 2), its own half of the scores, its own P buffer and its own accumulator,
-//                maximum and sum, so the groups never wait for one another before the end.
+//                j = g (mod 2), its own P buffer, accumulator, maximum and sum, so the groups never wait
+//                for one another before the end.
 // A group's accumulator is rescaled only when a row's maximum has grown by more than 2^8; weights are
 // relative to the maximum of the last rescaling, so they stay below 2^8.  A weight enters the P.V product
 // as the sum of two bf16 numbers.  At the end the two accumulators and the sink are merged.
@@ -53,10 +54,24 @@ struct Layout {  // of the shared memory, in bytes from a 1024-byte boundary
 };
 
 struct Bars {
-    uint64_t q_full, q_ready, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], o_done[2];
+    uint64_t q_full, q_ready, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[4], p_full[2], o_done[2];
     uint32_t tmem;
     int abort;
 };
+
+// A wait in the chain from one tile to the next: polls first, then the timed wait.
+__device__ __forceinline__ bool wait_soon(uint64_t *bar, uint32_t parity, volatile int *abort_flag, tlc_dev_status *status, int where,
+                                          uint64_t wait_ns) {
+    for (int i = 0; i < 64; i++)
+        if (tlc_gemm::mbar_try_wait(bar, parity)) return true;
+    return mbar_wait(bar, parity, abort_flag, status, where, wait_ns);
+}
+// 2^x; results below the normal numbers are zero.
+__device__ __forceinline__ float exp2_ftz(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
     asm volatile(
@@ -95,6 +110,7 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
             mbar_init(&b->v_full[s], 1);
             mbar_init(&b->v_empty[s], 1);
             mbar_init(&b->s_full[s], 1);
+            mbar_init(&b->s_full[2 + s], 1);
             mbar_init(&b->p_full[s], kGroup);
             mbar_init(&b->o_done[s], 1);
         }
@@ -109,7 +125,8 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = b->tmem;
-    const uint32_t tm_s[2] = {tmem, tmem + kTile}, tm_o[2] = {tmem + 2 * kTile, tmem + 2 * kTile + (uint32_t)p.V};
+    const int ahead = 4 * kTile + 2 * p.V <= 512 ? 4 : 2;  // score buffers
+    const uint32_t tm_o[2] = {tmem + ahead * kTile, tmem + ahead * kTile + (uint32_t)p.V};
     pdl_enter();
 
     if (warp == 0) {
@@ -122,28 +139,34 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
                 for (int c = 0; c < lay.chunks_r; c++)
                     tma_load_2d(at + (lay.chunks_d + c) * kQChunk, p.q_map, x_q + p.D + 64 * c, row0, bar);
             }
-            int j = 0;
-            for (; j < n_tiles; j++) {
-                const int st = j & 1;
-                const uint32_t free_parity = ((j >> 1) & 1u) ^ 1u;
-                if (!mbar_wait(&b->k_empty[st], free_parity, abort_flag, p.status, 31, p.wait_ns)) break;
+            int nk = 0, nv = 0;  // tiles asked for
+            auto load_k = [&] {
+                const int st = nk & 1;
+                if (!mbar_wait(&b->k_empty[st], ((nk >> 1) & 1u) ^ 1u, abort_flag, p.status, 31, p.wait_ns)) return false;
                 mbar_arrive_expect_tx(&b->k_full[st], (uint32_t)lay.k_stage);
-                uint32_t at = smem_u32(base + lay.k + st * lay.k_stage), bar = smem_u32(&b->k_full[st]);
-                for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kKChunk, p.k_map, x_k + 64 * c, j * kTile, bar);
+                const uint32_t at = smem_u32(base + lay.k + st * lay.k_stage), bar = smem_u32(&b->k_full[st]);
+                for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kKChunk, p.k_map, x_k + 64 * c, nk * kTile, bar);
                 for (int c = 0; c < lay.chunks_r; c++)
-                    tma_load_2d(at + (lay.chunks_d + c) * kKChunk, p.rot_map, 64 * c, p.slot0 * p.max_seq + j * kTile, bar);
-                if (!mbar_wait(&b->v_empty[st], free_parity, abort_flag, p.status, 32, p.wait_ns)) break;
+                    tma_load_2d(at + (lay.chunks_d + c) * kKChunk, p.rot_map, 64 * c, p.slot0 * p.max_seq + nk * kTile, bar);
+                nk++;
+                return true;
+            };
+            auto load_v = [&] {
+                const int st = nv & 1;
+                if (!mbar_wait(&b->v_empty[st], ((nv >> 1) & 1u) ^ 1u, abort_flag, p.status, 32, p.wait_ns)) return false;
                 mbar_arrive_expect_tx(&b->v_full[st], (uint32_t)lay.v_stage);
-                at = smem_u32(base + lay.v + st * lay.v_stage);
-                bar = smem_u32(&b->v_full[st]);
-                for (int r = 0; r < lay.v_rows; r += 64) tma_load_2d(at + r * 128, p.v_map, j * kTile, head * p.V + r, bar);
-            }
+                const uint32_t at = smem_u32(base + lay.v + st * lay.v_stage), bar = smem_u32(&b->v_full[st]);
+                for (int r = 0; r < lay.v_rows; r += 64) tma_load_2d(at + r * 128, p.v_map, nv * kTile, head * p.V + r, bar);
+                nv++;
+                return true;
+            };
+            // keys two tiles ahead of the values: the scores of tile j + 3 come before P V of tile j
+            bool ok = load_k() && (n_tiles < 2 || load_k());
+            while (ok && nv < n_tiles) ok = load_v() && (nk == n_tiles || load_k());
             if (*abort_flag) {  // no copy may be in flight when the CTA ends
                 mbar_wait(&b->q_full, 0, abort_flag, p.status, 33, p.wait_ns);
-                for (int i = j - 2 > 0 ? j - 2 : 0; i <= j && i < n_tiles; i++) {
-                    mbar_wait(&b->k_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
-                    if (i < j) mbar_wait(&b->v_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
-                }
+                for (int i = nk > 2 ? nk - 2 : 0; i < nk; i++) mbar_wait(&b->k_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
+                for (int i = nv > 2 ? nv - 2 : 0; i < nv; i++) mbar_wait(&b->v_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
             }
         }
         __syncwarp();
@@ -151,29 +174,30 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
         if (lane == 0) {
             const uint32_t idesc_s = tlc_gemm::idesc_for(kTile) | kIdesc, idesc_o = tlc_gemm::idesc_for(p.V) | kIdesc;
             auto scores = [&](int j) {
-                const int st = j & 1;
-                if (!mbar_wait(&b->k_full[st], (j >> 1) & 1u, abort_flag, p.status, 34, p.wait_ns)) return false;
+                const int st = j & 1, buf = j & (ahead - 1);
+                const uint32_t to = tmem + buf * kTile;
+                if (!wait_soon(&b->k_full[st], (j >> 1) & 1u, abort_flag, p.status, 34, p.wait_ns)) return false;
                 tc_fence_after();
                 const uint32_t qa = smem_u32(base + lay.q), ka = smem_u32(base + lay.k + st * lay.k_stage);
                 for (int kk = 0; kk < p.D / 16; kk++)
-                    umma_f16(tm_s[st], make_desc(qa + (kk >> 2) * kQChunk + (kk & 3) * 32), make_desc(ka + (kk >> 2) * kKChunk + (kk & 3) * 32),
+                    umma_f16(to, make_desc(qa + (kk >> 2) * kQChunk + (kk & 3) * 32), make_desc(ka + (kk >> 2) * kKChunk + (kk & 3) * 32),
                              idesc_s, kk > 0 ? 1u : 0u);
                 for (int kk = 0; kk < p.R / 16; kk++)
-                    umma_f16(tm_s[st], make_desc(qa + (lay.chunks_d + (kk >> 2)) * kQChunk + (kk & 3) * 32),
+                    umma_f16(to, make_desc(qa + (lay.chunks_d + (kk >> 2)) * kQChunk + (kk & 3) * 32),
                              make_desc(ka + (lay.chunks_d + (kk >> 2)) * kKChunk + (kk & 3) * 32), idesc_s, 1u);
                 umma_commit(&b->k_empty[st]);
-                umma_commit(&b->s_full[st]);
+                umma_commit(&b->s_full[buf]);
                 return true;
             };
             bool ok = mbar_wait(&b->q_ready, 0, abort_flag, p.status, 35, p.wait_ns);
             tc_fence_after();
-            ok = ok && scores(0);
+            for (int j = 0; ok && j < ahead - 1 && j < n_tiles; j++) ok = scores(j);
             for (int j = 0; ok && j < n_tiles; j++) {
-                // the scores' buffer is free: its group has handed in the weights of tile j - 1
-                if (j + 1 < n_tiles && !scores(j + 1)) break;
+                // the buffer is free: its group has handed in the weights of tile j - 1
+                if (j + ahead - 1 < n_tiles && !scores(j + ahead - 1)) break;
                 const int g = j & 1;
-                if (!mbar_wait(&b->p_full[g], (j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
-                if (!mbar_wait(&b->v_full[g], (j >> 1) & 1u, abort_flag, p.status, 37, p.wait_ns)) break;
+                if (!wait_soon(&b->p_full[g], (j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
+                if (!wait_soon(&b->v_full[g], (j >> 1) & 1u, abort_flag, p.status, 37, p.wait_ns)) break;
                 tc_fence_after();
                 const uint32_t va = smem_u32(base + lay.v + g * lay.v_stage);
 #pragma unroll
@@ -216,11 +240,12 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
         uint8_t *ph = base + lay.p + (size_t)(2 * g) * kPBytes + r * 128, *pl = ph + kPBytes;
         int it = 0;
         for (int j = g; j < n_tiles; j += 2, it++) {
-            mbar_wait(&b->s_full[g], it & 1u, abort_flag, p.status, 39, p.wait_ns);
+            const int buf = j & (ahead - 1);
+            wait_soon(&b->s_full[buf], (ahead == 4 ? it >> 1 : it) & 1u, abort_flag, p.status, 39, p.wait_ns);
             tc_fence_after();
             uint32_t s[2][32];
-            tmem_ld32(tm_s[g] + lanes, s[0]);
-            tmem_ld32(tm_s[g] + lanes + 32, s[1]);
+            tmem_ld32(tmem + buf * kTile + lanes, s[0]);
+            tmem_ld32(tmem + buf * kTile + lanes + 32, s[1]);
             const int j0 = j * kTile;
             float mx0 = -INFINITY, mx1 = -INFINITY;
             if (j0 + kTile - 1 > warp_first) {  // some row of the warp does not see every key
@@ -235,22 +260,14 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
                 mx0 = fmaxf(mx0, __uint_as_float(s[0][e]));
                 mx1 = fmaxf(mx1, __uint_as_float(s[1][e]));
             }
-            // the smallest score stands for the maximum when the scale is negative: no assumption on its sign
-            float top = fmaxf(mx0, mx1) * scale2;
-            if (scale2 <= 0.f) {
-                top = -INFINITY;
-#pragma unroll
-                for (int e = 0; e < 32; e++) {
-                    if (j0 + e <= pos) top = fmaxf(top, __uint_as_float(s[0][e]) * scale2);
-                    if (j0 + 32 + e <= pos) top = fmaxf(top, __uint_as_float(s[1][e]) * scale2);
-                }
-            }
-            if (it > 0) mbar_wait(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
+            const float top = fmaxf(mx0, mx1) * scale2;  // the scale is positive
+            if (it > 0) wait_soon(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
             if (it == 0) {
                 m = top;
             } else if (__any_sync(0xffffffffu, top > m + 8.f)) {
                 const float m_new = fmaxf(m, top), f = m_new == -INFINITY ? 1.f : exp2f(m - m_new);
                 tc_fence_after();
+#pragma unroll 1
                 for (int c = 0; c < p.V; c += 16) {
                     uint32_t o[16];
                     tmem_ld16(tm_o[g] + lanes + c, o);
@@ -270,11 +287,7 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
                 for (int t = 0; t < 4; t++) {
                     const int e = 8 * (c & 3) + 2 * t;
                     const uint32_t *v = s[c >> 2];
-                    float a = exp2f(fmaf(__uint_as_float(v[e]), scale2, -from)), d = exp2f(fmaf(__uint_as_float(v[e + 1]), scale2, -from));
-                    if (scale2 <= 0.f) {
-                        a = j0 + 8 * c + 2 * t <= pos ? a : 0.f;
-                        d = j0 + 8 * c + 2 * t + 1 <= pos ? d : 0.f;
-                    }
+                    const float a = exp2_ftz(fmaf(__uint_as_float(v[e]), scale2, -from)), d = exp2_ftz(fmaf(__uint_as_float(v[e + 1]), scale2, -from));
                     sum0 += a;
                     sum1 += d;
                     split_pair(a, d, hi[t], lo[t]);
@@ -331,14 +344,14 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
 
 }  // namespace
 
-bool latent_prefill_fits(int D, int R, int V) {
+bool latent_prefill_fits(int D, int R, int V, float scale) {
     static_assert(sizeof(Bars) <= 256, "the barriers have 256 bytes");
-    return D % 16 == 0 && R % 16 == 0 && V % 16 == 0 && D > 0 && V > 0 && 2 * kTile + 2 * V <= 512 &&
+    return scale > 0.f && D % 16 == 0 && R % 16 == 0 && V % 16 == 0 && D > 0 && V > 0 && 2 * kTile + 2 * V <= 512 &&
            Layout(D, R, V).total + 1024 <= 227 * 1024;
 }
 
 int32_t launch_latent_prefill(tlc_ctx *ctx, const LatentParams &p) {
-    TLC_REQUIRE(latent_prefill_fits(p.D, p.R, p.V), TLC_ERR_INVALID_OPERATION, "latent attention: heads of %d + %d and %d values", p.D,
+    TLC_REQUIRE(latent_prefill_fits(p.D, p.R, p.V, p.scale), TLC_ERR_INVALID_OPERATION, "latent attention: heads of %d + %d and %d values", p.D,
                 p.R, p.V);
     static bool done[64] = {};
     if (!done[ctx->device & 63]) {
