@@ -3,13 +3,13 @@
 //
 // One CTA takes 128 queries of one head.  Keys come in tiles of 64: unrotated parts from k_all, the
 // rotated part all heads share straight from the cache, values transposed (V rows of 64 keys), so that
-// every operand is K-major; all by TMA with the 128-byte swizzle, two stages.
+// every operand is K-major; all by TMA with the 128-byte swizzle, two to four stages.
 //   warp 0       TMA
-//   warp 1       issues the MMAs: S = Q K^T runs up to three tiles ahead of P V (four score buffers; two
-//                when the accumulators leave no more room in the tensor memory)
+//   warp 1       issues the MMAs: S = Q K^T runs three tiles ahead of P V (four score buffers; one tile
+//                with two when the accumulators leave no more room in the tensor memory)
 //   warps 2-9    two softmax groups of 128 threads, one query row per thread; group g owns the tiles
-//                j = g (mod 2), its own P buffer, accumulator, maximum and sum, so the groups never wait
-//                for one another before the end.
+//                j = g (mod 2), its own accumulator, maximum and sum, so the groups never wait for one
+//                another before the end.  The weights P take the place of the scores in tensor memory.
 // A group's accumulator is rescaled only when a row's maximum has grown by more than 2^8; weights are
 // relative to the maximum of the last rescaling, so they stay below 2^8.  A weight enters the P.V product
 // as the sum of two bf16 numbers.  At the end the two accumulators and the sink are merged.
@@ -40,23 +40,40 @@ using tlc_gemm::umma_f16;
 constexpr int kRows = 128, kTile = 64;
 constexpr int kGroup = 128, kThreadsP = 64 + 2 * kGroup;
 constexpr int kQChunk = kRows * 128, kKChunk = kTile * 128;  // bytes of 64 columns
-constexpr int kPBytes = kRows * 128;                         // one part (high or low) of a group's weights
+constexpr int kMaxStages = 4;
 constexpr uint32_t kIdesc = (1u << 7) | (1u << 10);          // bf16 x bf16
 constexpr float kLog2e = 1.44269504088896340736f;
+constexpr size_t kSmemLimit = 226 * 1024, kExtra = 256 + 4 * kRows * sizeof(float);
 
 struct Layout {  // of the shared memory, in bytes from a 1024-byte boundary
-    int chunks_d, chunks_r, v_rows;
-    size_t k_stage, v_stage, q, k, v, p, bars, total;
+    int chunks_d, chunks_r, v_rows, stages;
+    size_t k_stage, v_stage, k, v, bars, total;
     __host__ __device__ Layout(int D, int R, int V)
         : chunks_d((D + 63) / 64), chunks_r((R + 63) / 64), v_rows((V + 63) / 64 * 64), k_stage((size_t)(chunks_d + chunks_r) * kKChunk),
-          v_stage((size_t)v_rows * 128), q(0), k(q + (size_t)(chunks_d + chunks_r) * kQChunk), v(k + 2 * k_stage), p(v + 2 * v_stage),
-          bars(p + 4 * (size_t)kPBytes), total(bars + 256 + 4 * kRows * sizeof(float)) {}
+          v_stage((size_t)v_rows * 128), k((size_t)(chunks_d + chunks_r) * kQChunk) {
+        const size_t room = kSmemLimit > k + kExtra ? kSmemLimit - k - kExtra : 0;
+        stages = (int)(room / (k_stage + v_stage));
+        if (stages > kMaxStages) stages = kMaxStages;
+        v = k + stages * k_stage;
+        bars = v + stages * v_stage;
+        total = bars + kExtra;
+    }
 };
 
 struct Bars {
-    uint64_t q_full, q_ready, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[4], p_full[2], o_done[2];
+    uint64_t q_full, q_ready, k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[4], p_full[4], o_done[2];
     uint32_t tmem;
     int abort;
+};
+struct Ring {  // position in a ring of stages
+    int at = 0;
+    uint32_t parity = 0;
+    __device__ __forceinline__ void next(int stages) {
+        if (++at == stages) {
+            at = 0;
+            parity ^= 1u;
+        }
+    }
 };
 
 // A wait in the chain from one tile to the next: polls first, then the timed wait.
@@ -90,6 +107,25 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 
+__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%32], "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,"
+        "%29,%30,%31};" ::"r"(r[0]),
+        "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
+        "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]),
+        "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]), "r"(taddr)
+        : "memory");
+}
+// D += A B with A (bf16, two values per 32-bit column, a row per lane) in tensor memory.
+__device__ __forceinline__ void umma_f16_tmem_a(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
+        " tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n" ::"r"(tmem_d),
+        "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+
 __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __grid_constant__ LatentParams p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t *base = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -104,16 +140,17 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
     if (tid == 0) {
         mbar_init(&b->q_full, 1);
         mbar_init(&b->q_ready, 2 * kGroup);
-        for (int s = 0; s < 2; s++) {
+        for (int s = 0; s < kMaxStages; s++) {
             mbar_init(&b->k_full[s], 1);
             mbar_init(&b->k_empty[s], 1);
             mbar_init(&b->v_full[s], 1);
             mbar_init(&b->v_empty[s], 1);
-            mbar_init(&b->s_full[s], 1);
-            mbar_init(&b->s_full[2 + s], 1);
-            mbar_init(&b->p_full[s], kGroup);
-            mbar_init(&b->o_done[s], 1);
         }
+        for (int s = 0; s < 4; s++) {
+            mbar_init(&b->s_full[s], 1);
+            mbar_init(&b->p_full[s], kGroup);
+        }
+        for (int s = 0; s < 2; s++) mbar_init(&b->o_done[s], 1);
         b->abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -134,81 +171,92 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
             const int x_q = head * (p.D + p.R), x_k = head * p.D;
             {
                 mbar_arrive_expect_tx(&b->q_full, (uint32_t)((lay.chunks_d + lay.chunks_r) * kQChunk));
-                const uint32_t at = smem_u32(base + lay.q), bar = smem_u32(&b->q_full);
+                const uint32_t at = smem_u32(base), bar = smem_u32(&b->q_full);
                 for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kQChunk, p.q_map, x_q + 64 * c, row0, bar);
                 for (int c = 0; c < lay.chunks_r; c++)
                     tma_load_2d(at + (lay.chunks_d + c) * kQChunk, p.q_map, x_q + p.D + 64 * c, row0, bar);
             }
             int nk = 0, nv = 0;  // tiles asked for
+            Ring rk, rv;
             auto load_k = [&] {
-                const int st = nk & 1;
-                if (!mbar_wait(&b->k_empty[st], ((nk >> 1) & 1u) ^ 1u, abort_flag, p.status, 31, p.wait_ns)) return false;
-                mbar_arrive_expect_tx(&b->k_full[st], (uint32_t)lay.k_stage);
-                const uint32_t at = smem_u32(base + lay.k + st * lay.k_stage), bar = smem_u32(&b->k_full[st]);
+                if (!mbar_wait(&b->k_empty[rk.at], rk.parity ^ 1u, abort_flag, p.status, 31, p.wait_ns)) return false;
+                mbar_arrive_expect_tx(&b->k_full[rk.at], (uint32_t)lay.k_stage);
+                const uint32_t at = smem_u32(base + lay.k + rk.at * lay.k_stage), bar = smem_u32(&b->k_full[rk.at]);
                 for (int c = 0; c < lay.chunks_d; c++) tma_load_2d(at + c * kKChunk, p.k_map, x_k + 64 * c, nk * kTile, bar);
                 for (int c = 0; c < lay.chunks_r; c++)
                     tma_load_2d(at + (lay.chunks_d + c) * kKChunk, p.rot_map, 64 * c, p.slot0 * p.max_seq + nk * kTile, bar);
                 nk++;
+                rk.next(lay.stages);
                 return true;
             };
             auto load_v = [&] {
-                const int st = nv & 1;
-                if (!mbar_wait(&b->v_empty[st], ((nv >> 1) & 1u) ^ 1u, abort_flag, p.status, 32, p.wait_ns)) return false;
-                mbar_arrive_expect_tx(&b->v_full[st], (uint32_t)lay.v_stage);
-                const uint32_t at = smem_u32(base + lay.v + st * lay.v_stage), bar = smem_u32(&b->v_full[st]);
+                if (!mbar_wait(&b->v_empty[rv.at], rv.parity ^ 1u, abort_flag, p.status, 32, p.wait_ns)) return false;
+                mbar_arrive_expect_tx(&b->v_full[rv.at], (uint32_t)lay.v_stage);
+                const uint32_t at = smem_u32(base + lay.v + rv.at * lay.v_stage), bar = smem_u32(&b->v_full[rv.at]);
                 for (int r = 0; r < lay.v_rows; r += 64) tma_load_2d(at + r * 128, p.v_map, nv * kTile, head * p.V + r, bar);
                 nv++;
+                rv.next(lay.stages);
                 return true;
             };
-            // keys two tiles ahead of the values: the scores of tile j + 3 come before P V of tile j
+            // keys two tiles ahead of the values: the scores of tile j + 3 come before P V of tile j + 1
             bool ok = load_k() && (n_tiles < 2 || load_k());
             while (ok && nv < n_tiles) ok = load_v() && (nk == n_tiles || load_k());
-            if (*abort_flag) {  // no copy may be in flight when the CTA ends
+            if (*abort_flag) {  // no copy may be in flight when the CTA ends: the last ones of every stage
                 mbar_wait(&b->q_full, 0, abort_flag, p.status, 33, p.wait_ns);
-                for (int i = nk > 2 ? nk - 2 : 0; i < nk; i++) mbar_wait(&b->k_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
-                for (int i = nv > 2 ? nv - 2 : 0; i < nv; i++) mbar_wait(&b->v_full[i & 1], (i >> 1) & 1u, abort_flag, p.status, 33, p.wait_ns);
+                for (int i = nk > lay.stages ? nk - lay.stages : 0; i < nk; i++)
+                    mbar_wait(&b->k_full[i % lay.stages], (i / lay.stages) & 1u, abort_flag, p.status, 33, p.wait_ns);
+                for (int i = nv > lay.stages ? nv - lay.stages : 0; i < nv; i++)
+                    mbar_wait(&b->v_full[i % lay.stages], (i / lay.stages) & 1u, abort_flag, p.status, 33, p.wait_ns);
             }
         }
         __syncwarp();
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t idesc_s = tlc_gemm::idesc_for(kTile) | kIdesc, idesc_o = tlc_gemm::idesc_for(p.V) | kIdesc;
+            Ring rk, rv;
+            const uint32_t qa = smem_u32(base);
             auto scores = [&](int j) {
-                const int st = j & 1, buf = j & (ahead - 1);
+                const int buf = j & (ahead - 1);
                 const uint32_t to = tmem + buf * kTile;
-                if (!wait_soon(&b->k_full[st], (j >> 1) & 1u, abort_flag, p.status, 34, p.wait_ns)) return false;
+                if (!wait_soon(&b->k_full[rk.at], rk.parity, abort_flag, p.status, 34, p.wait_ns)) return false;
                 tc_fence_after();
-                const uint32_t qa = smem_u32(base + lay.q), ka = smem_u32(base + lay.k + st * lay.k_stage);
+                const uint32_t ka = smem_u32(base + lay.k + rk.at * lay.k_stage);
                 for (int kk = 0; kk < p.D / 16; kk++)
                     umma_f16(to, make_desc(qa + (kk >> 2) * kQChunk + (kk & 3) * 32), make_desc(ka + (kk >> 2) * kKChunk + (kk & 3) * 32),
                              idesc_s, kk > 0 ? 1u : 0u);
                 for (int kk = 0; kk < p.R / 16; kk++)
                     umma_f16(to, make_desc(qa + (lay.chunks_d + (kk >> 2)) * kQChunk + (kk & 3) * 32),
                              make_desc(ka + (lay.chunks_d + (kk >> 2)) * kKChunk + (kk & 3) * 32), idesc_s, 1u);
-                umma_commit(&b->k_empty[st]);
+                umma_commit(&b->k_empty[rk.at]);
                 umma_commit(&b->s_full[buf]);
+                rk.next(lay.stages);
                 return true;
             };
             bool ok = mbar_wait(&b->q_ready, 0, abort_flag, p.status, 35, p.wait_ns);
             tc_fence_after();
             for (int j = 0; ok && j < ahead - 1 && j < n_tiles; j++) ok = scores(j);
             for (int j = 0; ok && j < n_tiles; j++) {
-                // the buffer is free: its group has handed in the weights of tile j - 1
-                if (j + ahead - 1 < n_tiles && !scores(j + ahead - 1)) break;
-                const int g = j & 1;
-                if (!wait_soon(&b->p_full[g], (j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
-                if (!wait_soon(&b->v_full[g], (j >> 1) & 1u, abort_flag, p.status, 37, p.wait_ns)) break;
+                const int g = j & 1, buf = j & (ahead - 1);
+                const uint32_t pa = tmem + buf * kTile;
+                if (!wait_soon(&b->p_full[buf], (ahead == 4 ? j >> 2 : j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
+                if (!wait_soon(&b->v_full[rv.at], rv.parity, abort_flag, p.status, 37, p.wait_ns)) break;
                 tc_fence_after();
-                const uint32_t va = smem_u32(base + lay.v + g * lay.v_stage);
+                const uint32_t va = smem_u32(base + lay.v + rv.at * lay.v_stage);
 #pragma unroll
-                for (int part = 0; part < 2; part++) {
-                    const uint32_t pa = smem_u32(base + lay.p + (size_t)(2 * g + part) * kPBytes);
+                for (int part = 0; part < 2; part++)
 #pragma unroll
                     for (int kk = 0; kk < kTile / 16; kk++)
-                        umma_f16(tm_o[g], make_desc(pa + kk * 32), make_desc(va + kk * 32), idesc_o, j > 1 || part > 0 || kk > 0 ? 1u : 0u);
-                }
-                umma_commit(&b->v_empty[g]);
+                        umma_f16_tmem_a(tm_o[g], pa + part * (kTile / 2) + kk * 8, make_desc(va + kk * 32), idesc_o,
+                                        j > 1 || part > 0 || kk > 0 ? 1u : 0u);
+                umma_commit(&b->v_empty[rv.at]);
                 umma_commit(&b->o_done[g]);
+                rv.next(lay.stages);
+                // The scores' buffer held the weights of tile j - 1: that product, of another shape and hence not
+                // ordered with this one, must be complete.
+                if (j + ahead - 1 < n_tiles) {
+                    if (j > 0 && !wait_soon(&b->o_done[g ^ 1], ((j - 1) >> 1) & 1u, abort_flag, p.status, 42, p.wait_ns)) break;
+                    if (!scores(j + ahead - 1)) break;
+                }
             }
         }
         __syncwarp();
@@ -220,7 +268,7 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
         mbar_wait(&b->q_full, 0, abort_flag, p.status, 38, p.wait_ns);
         for (int i = 4 * g; i < p.R / 2; i += 8) {  // four pairs: one 16-byte piece
             const int e = 2 * i, c = e >> 6, piece = (e & 63) >> 3;
-            uint4 *at = reinterpret_cast<uint4 *>(base + lay.q + (size_t)(lay.chunks_d + c) * kQChunk + r * 128 + ((piece ^ (r & 7)) << 4));
+            uint4 *at = reinterpret_cast<uint4 *>(base + (size_t)(lay.chunks_d + c) * kQChunk + r * 128 + ((piece ^ (r & 7)) << 4));
             float f[8];
             unpack(*at, f);
             uint32_t o[4];
@@ -237,7 +285,6 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
 
         const float scale2 = p.scale * kLog2e;
         float m = -INFINITY, l = 0.f;
-        uint8_t *ph = base + lay.p + (size_t)(2 * g) * kPBytes + r * 128, *pl = ph + kPBytes;
         int it = 0;
         for (int j = g; j < n_tiles; j += 2, it++) {
             const int buf = j & (ahead - 1);
@@ -261,10 +308,10 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
                 mx1 = fmaxf(mx1, __uint_as_float(s[1][e]));
             }
             const float top = fmaxf(mx0, mx1) * scale2;  // the scale is positive
-            if (it > 0) wait_soon(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
             if (it == 0) {
                 m = top;
             } else if (__any_sync(0xffffffffu, top > m + 8.f)) {
+                wait_soon(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
                 const float m_new = fmaxf(m, top), f = m_new == -INFINITY ? 1.f : exp2f(m - m_new);
                 tc_fence_after();
 #pragma unroll 1
@@ -280,25 +327,24 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
             }
             const float from = m == -INFINITY ? 0.f : m;
             float sum0 = 0.f, sum1 = 0.f;
+            uint32_t hi[32], lo[32];
 #pragma unroll
-            for (int c = 0; c < 8; c++) {  // eight keys: one 16-byte piece of each part
-                uint32_t hi[4], lo[4];
+            for (int c = 0; c < 2; c++) {
 #pragma unroll
-                for (int t = 0; t < 4; t++) {
-                    const int e = 8 * (c & 3) + 2 * t;
-                    const uint32_t *v = s[c >> 2];
-                    const float a = exp2_ftz(fmaf(__uint_as_float(v[e]), scale2, -from)), d = exp2_ftz(fmaf(__uint_as_float(v[e + 1]), scale2, -from));
+                for (int e = 0; e < 32; e += 2) {
+                    const float a = exp2_ftz(fmaf(__uint_as_float(s[c][e]), scale2, -from));
+                    const float d = exp2_ftz(fmaf(__uint_as_float(s[c][e + 1]), scale2, -from));
                     sum0 += a;
                     sum1 += d;
-                    split_pair(a, d, hi[t], lo[t]);
+                    split_pair(a, d, hi[16 * c + e / 2], lo[16 * c + e / 2]);
                 }
-                *reinterpret_cast<uint4 *>(ph + ((c ^ (r & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                *reinterpret_cast<uint4 *>(pl + ((c ^ (r & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
             }
+            tmem_st32(tmem + buf * kTile + lanes, hi);
+            tmem_st32(tmem + buf * kTile + lanes + kTile / 2, lo);
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             l += sum0 + sum1;
-            fence_async_proxy();
             tc_fence_before();
-            mbar_arrive(&b->p_full[g]);
+            mbar_arrive(&b->p_full[buf]);
         }
         if (it > 0) mbar_wait(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 41, p.wait_ns);
         stat[g * kRows + r] = m;
@@ -346,8 +392,8 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
 
 bool latent_prefill_fits(int D, int R, int V, float scale) {
     static_assert(sizeof(Bars) <= 256, "the barriers have 256 bytes");
-    return scale > 0.f && D % 16 == 0 && R % 16 == 0 && V % 16 == 0 && D > 0 && V > 0 && 2 * kTile + 2 * V <= 512 &&
-           Layout(D, R, V).total + 1024 <= 227 * 1024;
+    return scale > 0.f && D % 16 == 0 && R % 16 == 0 && V % 16 == 0 && D > 0 && V > 0 && 2 * kTile + 2 * V <= 512 && D + R <= 512 &&
+           Layout(D, R, V).stages >= 2;
 }
 
 int32_t launch_latent_prefill(tlc_ctx *ctx, const LatentParams &p) {
