@@ -400,7 +400,7 @@ struct LatentParams {
     void *cache;              // T [slot][max_seq][row]
     const int *pos, *slot;
     void *ql;                 // T [m][H][row]: absorbed queries
-    float *part, *stat;       // [m][nsplit][H][kp]; [m][nsplit][H][2]: maximum (base 2) and sum
+    float *part, *stat;       // [m][nsplit][H][kp]; [m][H][nsplit][2]: maximum (base 2) and sum
     int nsplit;
     void *out;                // T [m][ldo], head h at h * V
     int ldo;

@@ -24,9 +24,11 @@ namespace tlc_dense {
 
 namespace {
 
-constexpr int kQueryThreads = 512, kScanThreads = 256, kScanWarps = kScanThreads / 32, kValueThreads = 512;
+constexpr int kQueryThreads = 512, kScanThreads = 512, kValueThreads = 512;
 constexpr int kKeys = 64;       // keys per tile
 constexpr int kTileHeads = 16;
+constexpr int kMaxSplits = 64;
+constexpr size_t kScanSmem = 216 * 1024;  // dynamic; the scores and factors of a tile come on top
 constexpr int kPPitch = kKeys + 8;
 constexpr float kLog2e = 1.44269504088896340736f;
 
@@ -110,9 +112,10 @@ __device__ __forceinline__ void store_remote_f32(float *at, int rank, float v) {
 
 // Grid (C, H [+ 1: the append], rows); the C CTAs of a head are a cluster when p.q is null.
 template <typename T>
-__global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __grid_constant__ LatentParams p, int split) {
+__global__ void __launch_bounds__(kQueryThreads, 2) latent_query_kernel(const __grid_constant__ LatentParams p, int split) {
     constexpr int N = Vec<T>::N, KEPT = 4;
     extern __shared__ __align__(16) float smem[];
+    __shared__ float red[33];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, C = gridDim.x, rank = blockIdx.x, head = blockIdx.y,
               r = blockIdx.z;
     if (head == p.H) {
@@ -138,25 +141,44 @@ __global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __
     // weights are never written: they can be on their way before the input exists
     if (!p.q)
         for (int i = lo + tid; i < hi; i += kQueryThreads) prefetch_l2(uq + (size_t)i * p.uq_pitch, (uint32_t)(qpieces * 16));
+    if (p_hi > p_lo)
+        for (int i = tid; i < p.D; i += kQueryThreads) prefetch_l2(uk + (size_t)i * p.uk_pitch + p_lo * N, (uint32_t)((p_hi - p_lo) * 16));
+    float sn = 0.f, cs = 1.f;  // of pair `tid` (more pairs than threads: made where they are used)
+    if (rank == 0 && 2 * tid < p.R) sincosf((float)pos * p.freq[tid], &sn, &cs);
     uint4 kept[KEPT];
+    auto keep = [&] {  // the first rows of W_uk, on their way while the CTAs exchange the query
 #pragma unroll
-    for (int i = 0; i < KEPT; i++)
-        kept[i] = g < groups && g + i * groups < p.D ? load_weight(reinterpret_cast<const uint4 *>(uk + (size_t)(g + i * groups) * p.uk_pitch) + c_own)
-                                                     : make_uint4(0u, 0u, 0u, 0u);
+        for (int i = 0; i < KEPT; i++)
+            kept[i] = g < groups && g + i * groups < p.D
+                          ? load_weight(reinterpret_cast<const uint4 *>(uk + (size_t)(g + i * groups) * p.uk_pitch) + c_own)
+                          : make_uint4(0u, 0u, 0u, 0u);
+    };
     pdl_enter();
     if (p.q) {
+        keep();
         const T *q = static_cast<const T *>(p.q) + (size_t)r * p.ldq + (size_t)head * DR;
         for (int i = tid; i < DR; i += kQueryThreads) qs[i] = to_f32(q[i]);
         __syncthreads();
     } else {
         const T *z = static_cast<const T *>(p.cq_raw) + (size_t)r * p.ldcq;
-        const float rstd = warp_rms(z, p.QR, p.eps, lane);  // every warp by itself
-        for (int c = tid; c < qpieces; c += kQueryThreads) {
-            float f[N], w[N];
+        float s = 0.f;
+        for (int c = tid; c < qpieces; c += kQueryThreads) {  // rows are padded to whole pieces, with anything
+            float f[N];
             unpack(__ldcg(reinterpret_cast<const uint4 *>(z) + c), f);
+#pragma unroll
+            for (int e = 0; e < N; e++) {
+                if (N * c + e >= p.QR) f[e] = 0.f;
+                s += f[e] * f[e];
+            }
+            put_piece<T>(cq, c, qpieces, f);
+        }
+        const float rstd = 1.0f / sqrtf(block_sum(s, red) / (float)p.QR + p.eps);
+        for (int c = tid; c < qpieces; c += kQueryThreads) {  // the thread's own pieces
+            float f[N], w[N];
+            get_piece<T>(cq, c, qpieces, f);
             unpack(load_nc(static_cast<const T *>(p.dq_norm) + c * N), w);
 #pragma unroll
-            for (int e = 0; e < N; e++) f[e] = N * c + e < p.QR ? f[e] * rstd * w[e] : 0.f;
+            for (int e = 0; e < N; e++) f[e] *= rstd * w[e];
             put_piece<T>(cq, c, qpieces, f);
         }
         __syncthreads();
@@ -171,6 +193,7 @@ __global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __
                 it.scale = 1.f;
                 return it;
             });
+        keep();
         __syncthreads();
         if (cluster) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");  // every peer is running
         for (int i = tid; i < (hi - lo) * C; i += kQueryThreads) {
@@ -194,7 +217,10 @@ __global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __
         for (int i = pieces * N + tid; i < p.kp; i += kQueryThreads) out[i] = from_f32<T>(0.f);
         for (int i = tid; i < (p.row - p.kp) / 2; i += kQueryThreads) {
             float2 v = make_float2(0.f, 0.f);
-            if (2 * i < p.R) v = rotate_pair(qs[p.D + 2 * i], qs[p.D + 2 * i + 1], pos, p.freq[i]);
+            if (2 * i < p.R) {
+                const float u = qs[p.D + 2 * i], w = qs[p.D + 2 * i + 1];
+                v = i == tid ? make_float2(u * cs - w * sn, w * cs + u * sn) : rotate_pair(u, w, pos, p.freq[i]);
+            }
             out[p.kp + 2 * i] = from_f32<T>(v.x);
             out[p.kp + 2 * i + 1] = from_f32<T>(v.y);
         }
@@ -225,10 +251,26 @@ __global__ void __launch_bounds__(kQueryThreads, 1) latent_query_kernel(const __
         for (int e = 0; e < N; e += 4)
             *reinterpret_cast<float4 *>(sums + tid * N + e) = make_float4(acc[e], acc[e + 1], acc[e + 2], acc[e + 3]);
         __syncthreads();
-        for (int i = tid; i < width * N; i += kQueryThreads) {
+        // `parts` threads per column, each every parts-th group, then one
+        const int columns = width * N, parts = columns < kQueryThreads ? kQueryThreads / columns : 1;
+        if (parts > 1) {
+            const int part = tid / columns, i = tid - part * columns;
             float a = 0.f;
-            for (int j = 0; j < groups; j++) a += sums[(size_t)j * np * N + i];
-            out[c0 * N + i] = from_f32<T>(a);
+            if (part < parts)
+                for (int j = part; j < groups; j += parts) a += sums[(size_t)j * np * N + i];
+            __syncthreads();
+            sums[tid] = a;
+            __syncthreads();
+            if (tid < columns) {
+                for (int j = 1; j < parts; j++) a += sums[j * columns + tid];
+                out[c0 * N + tid] = from_f32<T>(a);
+            }
+        } else {
+            for (int i = tid; i < columns; i += kQueryThreads) {
+                float a = 0.f;
+                for (int j = 0; j < groups; j++) a += sums[(size_t)j * np * N + i];
+                out[c0 * N + i] = from_f32<T>(a);
+            }
         }
         __syncthreads();
     }
@@ -258,8 +300,8 @@ __host__ __device__ constexpr size_t scan_smem(int row, int stages) {
     return (size_t)(stages * kKeys + kTileHeads) * scan_pitch(row) * 2 + (size_t)2 * kTileHeads * kPPitch * 2;
 }
 
-// Grid (nsplit, 16-head tiles, rows).  Eight warps: eight keys each for the scores, 8 NT columns each for
-// the weighted sum.
+// Grid (nsplit, 16-head tiles, rows).  Sixteen warps.  Scores: warp w takes eight keys (w mod 8) and half of the
+// columns; softmax: warp w takes head w; weighted sum: warp w takes 8 NT columns.
 template <int NT>
 __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_constant__ LatentParams p) {
     extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -267,7 +309,7 @@ __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_
     bf16 *ks = reinterpret_cast<bf16 *>(smem_raw);  // [2][64][pitch]
     bf16 *qs = ks + 2 * tile_elems;                 // [16][pitch]
     bf16 *ph = qs + kTileHeads * pitch, *pl = ph + kTileHeads * kPPitch;
-    __shared__ float wmax[kScanWarps][kTileHeads], wsum[kScanWarps][kTileHeads];
+    __shared__ float sc[2][kTileHeads][kKeys + 2], corr[kTileHeads];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3, mi = lane >> 3;
     const int split = blockIdx.x, head0 = blockIdx.y * kTileHeads, r = blockIdx.z;
     const int heads = p.H - head0 < kTileHeads ? p.H - head0 : kTileHeads;
@@ -298,12 +340,13 @@ __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_
     }
     if (st.lo < st.hi) load_tile(st.lo, 0, early, kKeys);
     cp_async_commit();
-    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    float m_run = -INFINITY, l_run = 0.f;  // of head `warp`
     float o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const float scale2 = p.scale * kLog2e;
-    const int ksteps = (pitch - 8) / 16, col0 = warp * 8 * NT;
+    const int kpairs = (pitch - 8) / 32, half = warp >> 3, k_lo = half ? (kpairs + 1) / 2 : 0, k_hi = half ? kpairs : (kpairs + 1) / 2;
+    const int col0 = warp * 8 * NT;
     for (int tile = st.lo; tile < st.hi; tile++) {
         const int stage = (tile - st.lo) & 1;
         if (tile + 1 < st.hi) {
@@ -317,54 +360,46 @@ __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_
         const bf16 *kt = ks + stage * tile_elems;
         float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
         const bf16 *qa_at = qs + ((mi & 1) * 8 + (lane & 7)) * pitch + (mi >> 1) * 8;
-        const bf16 *kb_at = kt + (8 * warp + (lane & 7)) * pitch + mi * 8;
-#pragma unroll 2
-        for (int kk = 0; kk < ksteps; kk += 2) {
+        const bf16 *kb_at = kt + (8 * (warp & 7) + (lane & 7)) * pitch + mi * 8;
+#pragma unroll 3
+        for (int kk = k_lo; kk < k_hi; kk++) {
             uint32_t a0[4], a1[4], b[4];
-            ldsm_x4(a0, qa_at + 16 * kk);
-            ldsm_x4(a1, qa_at + 16 * kk + 16);
-            ldsm_x4(b, kb_at + 16 * kk);
+            ldsm_x4(a0, qa_at + 32 * kk);
+            ldsm_x4(a1, qa_at + 32 * kk + 16);
+            ldsm_x4(b, kb_at + 32 * kk);
             mma_bf16(s, a0, b[0], b[1]);
             mma_bf16(s2, a1, b[2], b[3]);
         }
-        float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int j = tile * kKeys + 8 * warp + 2 * t + (e & 1);
-            s[e] = j < keys ? (s[e] + s2[e]) * scale2 : -INFINITY;
-            mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
-        }
-#pragma unroll
-        for (int h = 0; h < 2; h++) {
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-            if (t == 0) wmax[warp][g + 8 * h] = mx[h];
-        }
+        for (int h = 0; h < 2; h++)
+            *reinterpret_cast<float2 *>(&sc[half][g + 8 * h][8 * (warp & 7) + 2 * t]) = make_float2(s[2 * h] + s2[2 * h], s[2 * h + 1] + s2[2 * h + 1]);
         __syncthreads();
-        float corr[2];
+        {
+            const float2 u = *reinterpret_cast<const float2 *>(&sc[0][warp][2 * lane]), v = *reinterpret_cast<const float2 *>(&sc[1][warp][2 * lane]);
+            const int j = tile * kKeys + 2 * lane;
+            const float x = j < keys ? (u.x + v.x) * scale2 : -INFINITY, y = j + 1 < keys ? (u.y + v.y) * scale2 : -INFINITY;
+            float m = fmaxf(x, y);
 #pragma unroll
-        for (int h = 0; h < 2; h++) {
-            float m = m_run[h];
-#pragma unroll
-            for (int w = 0; w < kScanWarps; w++) m = fmaxf(m, wmax[w][g + 8 * h]);
-            corr[h] = exp2f(m_run[h] - m);  // a tile has at least one key: m is finite
-            m_run[h] = m;
-            const float a = exp2f(s[2 * h] - m), b = exp2f(s[2 * h + 1] - m);
-            l_run[h] = l_run[h] * corr[h] + a + b;
+            for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
+            m = fmaxf(m, m_run);  // a tile has at least one key: m is finite
+            const float c = exp2f(m_run - m), a = exp2f(x - m), b = exp2f(y - m);
+            m_run = m;
+            l_run = l_run * c + a + b;
             uint32_t hi, lo;
             split_pair(a, b, hi, lo);
-            const int at = (g + 8 * h) * kPPitch + 8 * warp + 2 * t;
-            *reinterpret_cast<uint32_t *>(ph + at) = hi;
-            *reinterpret_cast<uint32_t *>(pl + at) = lo;
-        }
-#pragma unroll
-        for (int d = 0; d < NT; d++) {
-            o[d][0] *= corr[0];
-            o[d][1] *= corr[0];
-            o[d][2] *= corr[1];
-            o[d][3] *= corr[1];
+            *reinterpret_cast<uint32_t *>(ph + warp * kPPitch + 2 * lane) = hi;
+            *reinterpret_cast<uint32_t *>(pl + warp * kPPitch + 2 * lane) = lo;
+            if (lane == 0) corr[warp] = c;
         }
         __syncthreads();
+        const float c0 = corr[g], c1 = corr[g + 8];
+#pragma unroll
+        for (int d = 0; d < NT; d++) {
+            o[d][0] *= c0;
+            o[d][1] *= c0;
+            o[d][2] *= c1;
+            o[d][3] *= c1;
+        }
 #pragma unroll
         for (int kk = 0; kk < kKeys / 16; kk++) {
             uint32_t hi[4], lo[4];
@@ -385,11 +420,11 @@ __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_
         __syncthreads();
     }
     cp_async_wait<0>();
+    l_run = warp_sum(l_run);
+    if (lane == 0 && warp < heads)
+        reinterpret_cast<float2 *>(p.stat)[((size_t)r * p.H + head0 + warp) * p.nsplit + split] = make_float2(m_run, l_run);
 #pragma unroll
     for (int h = 0; h < 2; h++) {
-        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
-        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
-        if (t == 0) wsum[warp][g + 8 * h] = l_run[h];
         const int row = g + 8 * h;
         if (row >= heads) continue;
         float *out = p.part + (((size_t)r * p.nsplit + split) * p.H + head0 + row) * p.kp;
@@ -398,14 +433,6 @@ __global__ void __launch_bounds__(kScanThreads) latent_scan_kernel(const __grid_
             const int c = col0 + 8 * d + 2 * t;
             if (c < p.kp) *reinterpret_cast<float2 *>(out + c) = make_float2(o[d][2 * h], o[d][2 * h + 1]);
         }
-        if (warp == 0 && t == 0) p.stat[(((size_t)r * p.nsplit + split) * p.H + head0 + row) * 2] = m_run[h];
-    }
-    __syncthreads();
-    if (tid < heads) {
-        float l = 0.f;
-#pragma unroll
-        for (int w = 0; w < kScanWarps; w++) l += wsum[w][tid];
-        p.stat[(((size_t)r * p.nsplit + split) * p.H + head0 + tid) * 2 + 1] = l;
     }
 }
 
@@ -473,16 +500,13 @@ __global__ void __launch_bounds__(128) latent_scan_fma_kernel(const __grid_const
 #pragma unroll
     for (int i = 0; i < kFmaCols / 32; i++)
         if (32 * i + lane < cols) p.part[at * p.kp + c0 + 32 * i + lane] = acc[i];
-    if (lane == 0 && c0 == 0) {
-        p.stat[2 * at] = m_run;
-        p.stat[2 * at + 1] = l_run;
-    }
+    if (lane == 0 && c0 == 0) reinterpret_cast<float2 *>(p.stat)[((size_t)r * p.H + head) * p.nsplit + split] = make_float2(m_run, l_run);
 }
 
 // Grid (shares of the head's values, H, rows).
 template <typename T>
-__global__ void __launch_bounds__(kValueThreads, 1) latent_value_kernel(const __grid_constant__ LatentParams p) {
-    constexpr int N = Vec<T>::N, WARPS = kValueThreads / 32, KEPT = 2, PARTS = 8;
+__global__ void __launch_bounds__(kValueThreads, 2) latent_value_kernel(const __grid_constant__ LatentParams p) {
+    constexpr int N = Vec<T>::N, WARPS = kValueThreads / 32, KEPT = 2, PARTS = 4;
     extern __shared__ __align__(16) float smem[];
     float *ol = smem, *f = ol + p.kp, *sums = f + ((p.nsplit + 3) & ~3);  // the head's weighted latent; factors; [kValueThreads][4]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y, r = blockIdx.z;
@@ -502,7 +526,8 @@ __global__ void __launch_bounds__(kValueThreads, 1) latent_value_kernel(const __
     const float sink = to_f32(static_cast<const T *>(p.sink)[head]) * kLog2e;
     pdl_enter();
     if (lo >= hi) return;
-    const float *stat = p.stat + ((size_t)r * p.nsplit * p.H + head) * 2, *part = p.part + ((size_t)r * p.nsplit * p.H + head) * p.kp;
+    const float2 *stat = reinterpret_cast<const float2 *>(p.stat) + ((size_t)r * p.H + head) * p.nsplit;
+    const float *part = p.part + ((size_t)r * p.nsplit * p.H + head) * p.kp;
     const size_t step = (size_t)p.H * p.kp;
     // a thread adds four columns of every `groups`-th stretch
     const int quads = p.kp / 4 < kValueThreads ? p.kp / 4 : kValueThreads, groups = kValueThreads / quads, g = tid / quads;
@@ -511,17 +536,18 @@ __global__ void __launch_bounds__(kValueThreads, 1) latent_value_kernel(const __
     for (int i = 0; i < PARTS; i++)
         if (g < groups && g + i * groups < p.nsplit)
             v[i] = __ldcg(reinterpret_cast<const float4 *>(part + (g + i * groups) * step) + (tid - g * quads));
-    {  // factors: exp2(m_s - m) / (sum_s l_s exp2(m_s - m) + exp2(sink - m)); every warp makes them all
-        float m = sink;
-        for (int s = lane; s < p.nsplit; s += 32) m = fmaxf(m, __ldcg(stat + (size_t)s * p.H * 2));
+    if (warp == WARPS - 1) {  // factors: exp2(m_s - m) / (sum_s l_s exp2(m_s - m) + exp2(sink - m)); at most 64 stretches
+        float2 a = make_float2(-INFINITY, 0.f), b = a;
+        if (lane < p.nsplit) a = __ldcg(stat + lane);
+        if (lane + 32 < p.nsplit) b = __ldcg(stat + lane + 32);
+        float m = fmaxf(fmaxf(a.x, b.x), sink);
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-        float l = 0.f;
-        for (int s = lane; s < p.nsplit; s += 32)
-            l += exp2f(__ldcg(stat + (size_t)s * p.H * 2) - m) * __ldcg(stat + (size_t)s * p.H * 2 + 1);
-        l = warp_sum(l) + exp2f(sink - m);
-        if (warp == 0)
-            for (int s = lane; s < p.nsplit; s += 32) f[s] = exp2f(__ldcg(stat + (size_t)s * p.H * 2) - m) / l;
+        a.x = exp2f(a.x - m);
+        b.x = exp2f(b.x - m);
+        const float l = warp_sum(a.x * a.y + b.x * b.y) + exp2f(sink - m);
+        if (lane < p.nsplit) f[lane] = a.x / l;
+        if (lane + 32 < p.nsplit) f[lane + 32] = b.x / l;
     }
     __syncthreads();
     for (int q0 = 0; q0 < p.kp / 4; q0 += quads) {
@@ -598,7 +624,7 @@ int32_t launched(tlc_ctx *ctx, cudaError_t le) {
     return TLC_OK;
 }
 
-bool scan_on_tensor_cores(const LatentParams &p, size_t elem) { return elem == 2 && p.kp <= 512 && scan_smem(p.row, 2) <= 220 * 1024; }
+bool scan_on_tensor_cores(const LatentParams &p, size_t elem) { return elem == 2 && p.kp <= 512 && scan_smem(p.row, 2) <= kScanSmem; }
 
 template <typename K>
 int32_t allow_smem(K kernel, bool (&done)[64], int device, size_t bytes) {
@@ -611,7 +637,7 @@ int32_t allow_smem(K kernel, bool (&done)[64], int device, size_t bytes) {
 template <int NT>
 int32_t scan_t(tlc_ctx *ctx, const LatentParams &p) {
     static bool done[64] = {};
-    if (int32_t rc = allow_smem(latent_scan_kernel<NT>, done, ctx->device, 220 * 1024)) return rc;
+    if (int32_t rc = allow_smem(latent_scan_kernel<NT>, done, ctx->device, kScanSmem)) return rc;
     return launched(ctx, tlc_launch_pdl(ctx, latent_scan_kernel<NT>,
                                         dim3((unsigned)p.nsplit, (unsigned)((p.H + kTileHeads - 1) / kTileHeads), (unsigned)p.m),
                                         dim3(kScanThreads), scan_smem(p.row, 2), p));
@@ -623,7 +649,7 @@ int latent_splits(const tlc_ctx *ctx, const LatentParams &p) {
     const int per_row = (p.H + kTileHeads - 1) / kTileHeads, tiles = (p.max_seq + kKeys - 1) / kKeys;
     int n = ctx->sm_count / (per_row * p.m);
     n = n < tiles ? n : tiles;
-    return n < 1 ? 1 : n > 64 ? 64 : n;
+    return n < 1 ? 1 : n > kMaxSplits ? kMaxSplits : n;
 }
 
 template <typename T>
@@ -671,7 +697,7 @@ template <typename T>
 int32_t launch_latent_absorbed(tlc_ctx *ctx, const LatentParams &p) {
     int32_t rc;
     if (scan_on_tensor_cores(p, sizeof(T))) {
-        rc = p.kp <= 128 ? scan_t<2>(ctx, p) : p.kp <= 256 ? scan_t<4>(ctx, p) : scan_t<8>(ctx, p);
+        rc = p.kp <= 256 ? scan_t<2>(ctx, p) : scan_t<4>(ctx, p);
     } else {
         const size_t smem = (size_t)4 * p.row * sizeof(float);
         TLC_REQUIRE(smem <= 200 * 1024, TLC_ERR_INVALID_OPERATION, "latent attention: cache rows of %d values do not fit", p.row);
