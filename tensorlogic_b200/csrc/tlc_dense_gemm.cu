@@ -181,7 +181,7 @@ __device__ __forceinline__ void store_piece(const GemmGroup &g, const uint32_t (
 
 // 32 columns of the warp's 32 rows (lane = row of `acc`) into the residual streams.  Rows turn into
 // columns through shared memory, 16 columns at a time, so that four lanes share a row's 64 bytes and
-// the loads of all streams are in flight together.  The first `rows` of the 32 exist.
+// the loads of all streams are in flight together.  Rows from `rows` on (if below 32) do not exist.
 template <int MAXS>
 __device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsOut &st, const uint32_t (&acc)[32], float *turn,
                                               int row0, int rows, int nb, int lane) {
@@ -198,7 +198,7 @@ __device__ __forceinline__ void store_streams(const GemmGroup &g, const StreamsO
         const int n = nb + 16 * half + 4 * (lane & 3);
         if (n >= g.n) continue;
         if ((g.n & 3) != 0) {  // rows do not start on 16-byte boundaries
-            for (int i = lane >> 2; i < rows; i += 8)
+            for (int i = lane >> 2; i < rows && i < 32; i += 8)
                 for (int e = 0; e < 4 && n + e < g.n; e++)
                     streams_column<bf16>(st, row0 + i, g.n, n + e,
                                          turn[i * kTurnPitch + 4 * (lane & 3) + e] +

@@ -1,4 +1,4 @@
-"""Small configurations, random weights and files for the decoder tests."""
+"""Small configurations, random weights, files and ways to feed a runner for the decoder tests."""
 import json
 import struct
 
@@ -110,3 +110,32 @@ def error(got, want):
     d = d - d.mean(-1, keepdims=True)
     size = np.sqrt(((want - want.mean(-1, keepdims=True)) ** 2).mean())
     return float(np.sqrt((d * d).mean(-1)).max() / size)
+
+
+# ---- ways to feed a sequence to a runner -------------------------------------------------------------
+
+def whole(dec, seq):
+    s = dec.open()
+    out = dec.feed(s, seq, range(len(seq)))
+    dec.close(s)
+    return out
+
+
+def one_by_one(dec, seq, first=1):
+    s = dec.open()
+    rows = [dec.feed(s, seq[:first], range(first))]
+    rows += [dec.feed(s, [t], [0]) for t in seq[first:]]
+    dec.close(s)
+    return np.concatenate(rows)
+
+
+def portions(dec, seq, sizes):
+    s, at, rows = dec.open(), 0, []
+    for n in sizes:
+        part = seq[at:at + n]
+        if len(part):
+            rows.append(dec.feed(s, part, range(len(part))))
+        at += n
+    assert at >= len(seq)
+    dec.close(s)
+    return np.concatenate(rows)

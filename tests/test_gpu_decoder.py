@@ -10,7 +10,8 @@ import pytest
 
 import decoder_ref as ref
 from conftest import ROOT
-from decoder_util import attention, config, dense, error, moe, tokens, weights, write_model, write_safetensors
+from decoder_util import (attention, config, dense, error, moe, one_by_one, portions, tokens, weights, whole, write_model,
+                          write_safetensors)
 
 pytestmark = pytest.mark.gpu
 
@@ -23,33 +24,6 @@ def build(dev, cfg, w, dtype, **kw):
     from tensorlogic_b200.decoder import Decoder, model_from_arrays
     kw.setdefault("max_seq", 512)
     return Decoder(dev, model_from_arrays(dev, w, dtype), toposun.read_config(cfg), dtype, **kw)
-
-
-def whole(dec, seq):
-    s = dec.open()
-    out = dec.feed(s, seq, range(len(seq)))
-    dec.close(s)
-    return out
-
-
-def one_by_one(dec, seq, first=1):
-    s = dec.open()
-    rows = [dec.feed(s, seq[:first], range(first))]
-    rows += [dec.feed(s, [t], [0]) for t in seq[first:]]
-    dec.close(s)
-    return np.concatenate(rows)
-
-
-def portions(dec, seq, sizes):
-    s, at, rows = dec.open(), 0, []
-    for n in sizes:
-        part = seq[at:at + n]
-        if len(part):
-            rows.append(dec.feed(s, part, range(len(part))))
-        at += n
-    assert at >= len(seq)
-    dec.close(s)
-    return np.concatenate(rows)
 
 
 def check(dev, cfg, w, seq, dtypes=DTYPES, tol=1.0, **kw):
