@@ -5,11 +5,14 @@
 // rotated part all heads share straight from the cache, values transposed (V rows of 64 keys), so that
 // every operand is K-major; all by TMA with the 128-byte swizzle, two to four stages.
 //   warp 0       TMA
-//   warp 1       issues the MMAs: S = Q K^T runs three tiles ahead of P V (four score buffers; one tile
-//                with two when the accumulators leave no more room in the tensor memory)
-//   warps 2-9    two softmax groups of 128 threads, one query row per thread; group g owns the tiles
+//   warp 1       issues S = Q K^T, as far ahead as there are score buffers (four; two when the accumulators
+//                leave no more room in the tensor memory)
+//   warp 2       issues P V
+//   warps 3-10   two softmax groups of 128 threads, one query row per thread; group g owns the tiles
 //                j = g (mod 2), its own accumulator, maximum and sum, so the groups never wait for one
 //                another before the end.  The weights P take the place of the scores in tensor memory.
+// Issuing an MMA takes about as long as running one of this size: hence two issuing warps, each of
+// which runs its loop as a whole (descriptors in uniform registers) and elects the issuing thread.
 // A group's accumulator is rescaled only when a row's maximum has grown by more than 2^8; weights are
 // relative to the maximum of the last rescaling, so they stay below 2^8.  A weight enters the P.V product
 // as the sum of two bf16 numbers.  At the end the two accumulators and the sink are merged.
@@ -38,7 +41,7 @@ using tlc_gemm::umma_commit;
 using tlc_gemm::umma_f16;
 
 constexpr int kRows = 128, kTile = 64;
-constexpr int kGroup = 128, kThreadsP = 64 + 2 * kGroup;
+constexpr int kGroup = 128, kThreadsP = 96 + 2 * kGroup;
 constexpr int kQChunk = kRows * 128, kKChunk = kTile * 128;  // bytes of 64 columns
 constexpr int kMaxStages = 4;
 constexpr uint32_t kIdesc = (1u << 7) | (1u << 10);          // bf16 x bf16
@@ -61,7 +64,7 @@ struct Layout {  // of the shared memory, in bytes from a 1024-byte boundary
 };
 
 struct Bars {
-    uint64_t q_full, q_ready, k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[4], p_full[4], o_done[2];
+    uint64_t q_full, q_ready, k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[4], p_full[4], o_done[4];
     uint32_t tmem;
     int abort;
 };
@@ -82,6 +85,12 @@ __device__ __forceinline__ bool wait_soon(uint64_t *bar, uint32_t parity, volati
     for (int i = 0; i < 64; i++)
         if (tlc_gemm::mbar_try_wait(bar, parity)) return true;
     return mbar_wait(bar, parity, abort_flag, status, where, wait_ns);
+}
+// One thread of the warp.
+__device__ __forceinline__ bool elect_one() {
+    uint32_t p;
+    asm volatile("{\n .reg .pred q;\n elect.sync _|q, 0xffffffff;\n selp.u32 %0, 1, 0, q;\n}\n" : "=r"(p));
+    return p != 0;
 }
 // 2^x; results below the normal numbers are zero.
 __device__ __forceinline__ float exp2_ftz(float x) {
@@ -149,8 +158,8 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
         for (int s = 0; s < 4; s++) {
             mbar_init(&b->s_full[s], 1);
             mbar_init(&b->p_full[s], kGroup);
+            mbar_init(&b->o_done[s], 1);
         }
-        for (int s = 0; s < 2; s++) mbar_init(&b->o_done[s], 1);
         b->abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -198,7 +207,7 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
                 rv.next(lay.stages);
                 return true;
             };
-            // keys two tiles ahead of the values: the scores of tile j + 3 come before P V of tile j + 1
+            // keys two tiles ahead of the values, as their products
             bool ok = load_k() && (n_tiles < 2 || load_k());
             while (ok && nv < n_tiles) ok = load_v() && (nk == n_tiles || load_k());
             if (*abort_flag) {  // no copy may be in flight when the CTA ends: the last ones of every stage
@@ -211,57 +220,62 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
         }
         __syncwarp();
     } else if (warp == 1) {
-        if (lane == 0) {
-            const uint32_t idesc_s = tlc_gemm::idesc_for(kTile) | kIdesc, idesc_o = tlc_gemm::idesc_for(p.V) | kIdesc;
-            Ring rk, rv;
-            const uint32_t qa = smem_u32(base);
-            auto scores = [&](int j) {
-                const int buf = j & (ahead - 1);
-                const uint32_t to = tmem + buf * kTile;
-                if (!wait_soon(&b->k_full[rk.at], rk.parity, abort_flag, p.status, 34, p.wait_ns)) return false;
-                tc_fence_after();
-                const uint32_t ka = smem_u32(base + lay.k + rk.at * lay.k_stage);
-                for (int kk = 0; kk < p.D / 16; kk++)
-                    umma_f16(to, make_desc(qa + (kk >> 2) * kQChunk + (kk & 3) * 32), make_desc(ka + (kk >> 2) * kKChunk + (kk & 3) * 32),
-                             idesc_s, kk > 0 ? 1u : 0u);
-                for (int kk = 0; kk < p.R / 16; kk++)
-                    umma_f16(to, make_desc(qa + (lay.chunks_d + (kk >> 2)) * kQChunk + (kk & 3) * 32),
-                             make_desc(ka + (lay.chunks_d + (kk >> 2)) * kKChunk + (kk & 3) * 32), idesc_s, 1u);
-                umma_commit(&b->k_empty[rk.at]);
-                umma_commit(&b->s_full[buf]);
-                rk.next(lay.stages);
-                return true;
-            };
-            bool ok = mbar_wait(&b->q_ready, 0, abort_flag, p.status, 35, p.wait_ns);
+        const uint32_t idesc = tlc_gemm::idesc_for(kTile) | kIdesc;
+        const uint64_t qd = make_desc(smem_u32(base)), kd = make_desc(smem_u32(base + lay.k));
+        const uint32_t step = (uint32_t)(lay.k_stage >> 4);  // descriptors count 16 bytes
+        const int chunks = lay.chunks_d + lay.chunks_r;
+        Ring ring, bufs;
+        bool ok = mbar_wait(&b->q_ready, 0, abort_flag, p.status, 35, p.wait_ns);
+        for (int j = 0; j < n_tiles; j++) {
+            // the buffer held the weights of tile j - ahead: their product must be complete
+            if (j >= ahead) ok = ok && wait_soon(&b->o_done[bufs.at], bufs.parity ^ 1u, abort_flag, p.status, 42, p.wait_ns);
+            ok = ok && wait_soon(&b->k_full[ring.at], ring.parity, abort_flag, p.status, 34, p.wait_ns);
+            if (!__all_sync(0xffffffffu, ok)) break;
             tc_fence_after();
-            for (int j = 0; ok && j < ahead - 1 && j < n_tiles; j++) ok = scores(j);
-            for (int j = 0; ok && j < n_tiles; j++) {
-                const int g = j & 1, buf = j & (ahead - 1);
-                const uint32_t pa = tmem + buf * kTile;
-                if (!wait_soon(&b->p_full[buf], (ahead == 4 ? j >> 2 : j >> 1) & 1u, abort_flag, p.status, 36, p.wait_ns)) break;
-                if (!wait_soon(&b->v_full[rv.at], rv.parity, abort_flag, p.status, 37, p.wait_ns)) break;
-                tc_fence_after();
-                const uint32_t va = smem_u32(base + lay.v + rv.at * lay.v_stage);
+            const uint32_t to = tmem + bufs.at * kTile;
+            const uint64_t ks = kd + ring.at * step;
+            if (elect_one()) {
+                for (int c = 0; c < chunks; c++) {  // 64 columns: four steps of 16, fewer at the end of a part
+                    const int steps = c < lay.chunks_d ? p.D / 16 - 4 * c : p.R / 16 - 4 * (c - lay.chunks_d);
+                    const uint64_t qc = qd + c * (kQChunk >> 4), kc = ks + c * (kKChunk >> 4);
+                    umma_f16(to, qc, kc, idesc, c > 0 ? 1u : 0u);
 #pragma unroll
-                for (int part = 0; part < 2; part++)
-#pragma unroll
-                    for (int kk = 0; kk < kTile / 16; kk++)
-                        umma_f16_tmem_a(tm_o[g], pa + part * (kTile / 2) + kk * 8, make_desc(va + kk * 32), idesc_o,
-                                        j > 1 || part > 0 || kk > 0 ? 1u : 0u);
-                umma_commit(&b->v_empty[rv.at]);
-                umma_commit(&b->o_done[g]);
-                rv.next(lay.stages);
-                // The scores' buffer held the weights of tile j - 1: that product, of another shape and hence not
-                // ordered with this one, must be complete.
-                if (j + ahead - 1 < n_tiles) {
-                    if (j > 0 && !wait_soon(&b->o_done[g ^ 1], ((j - 1) >> 1) & 1u, abort_flag, p.status, 42, p.wait_ns)) break;
-                    if (!scores(j + ahead - 1)) break;
+                    for (int kk = 1; kk < 4; kk++)
+                        if (kk < steps) umma_f16(to, qc + 2 * kk, kc + 2 * kk, idesc, 1u);
                 }
+                umma_commit(&b->k_empty[ring.at]);
+                umma_commit(&b->s_full[bufs.at]);
             }
+            __syncwarp();
+            ring.next(lay.stages);
+            bufs.next(ahead);
         }
-        __syncwarp();
+    } else if (warp == 2) {
+        const uint32_t idesc = tlc_gemm::idesc_for(p.V) | kIdesc;
+        const uint64_t vd = make_desc(smem_u32(base + lay.v));
+        const uint32_t step = (uint32_t)(lay.v_stage >> 4);
+        Ring ring, bufs;
+        for (int j = 0; j < n_tiles; j++) {
+            const bool ok = wait_soon(&b->p_full[bufs.at], bufs.parity, abort_flag, p.status, 36, p.wait_ns) &&
+                            wait_soon(&b->v_full[ring.at], ring.parity, abort_flag, p.status, 37, p.wait_ns);
+            if (!__all_sync(0xffffffffu, ok)) break;
+            tc_fence_after();
+            const uint32_t pa = tmem + bufs.at * kTile, to = tmem + ahead * kTile + (j & 1) * p.V;
+            const uint64_t vs = vd + ring.at * step;
+            if (elect_one()) {
+                umma_f16_tmem_a(to, pa, vs, idesc, j > 1 ? 1u : 0u);
+#pragma unroll
+                for (int i = 1; i < kTile / 8; i++)  // the high parts of the weights, then the low ones
+                    umma_f16_tmem_a(to, pa + 8 * i, vs + 2 * (i & 3), idesc, 1u);
+                umma_commit(&b->v_empty[ring.at]);
+                umma_commit(&b->o_done[bufs.at]);
+            }
+            __syncwarp();
+            ring.next(lay.stages);
+            bufs.next(ahead);
+        }
     } else {
-        const int g = (warp - 2) >> 2, wq = warp & 3, r = 32 * wq + lane;  // tensor-memory lanes this warp may touch: 32 wq ..
+        const int g = (warp - 3) >> 2, wq = warp & 3, r = 32 * wq + lane;  // tensor-memory lanes this warp may touch: 32 wq ..
         const uint32_t lanes = (uint32_t)(32 * wq) << 16;
         const int pos = p.pos0 + row0 + r, warp_first = p.pos0 + row0 + 32 * wq;
         // rotate the queries: the groups share a row's pairs
@@ -285,10 +299,13 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
 
         const float scale2 = p.scale * kLog2e;
         float m = -INFINITY, l = 0.f;
+        // buffer and phase of a tile
+        auto buffer = [&](int j) { return j & (ahead - 1); };
+        auto phase = [&](int j) { return (uint32_t)(ahead == 4 ? j >> 2 : j >> 1) & 1u; };
         int it = 0;
         for (int j = g; j < n_tiles; j += 2, it++) {
-            const int buf = j & (ahead - 1);
-            wait_soon(&b->s_full[buf], (ahead == 4 ? it >> 1 : it) & 1u, abort_flag, p.status, 39, p.wait_ns);
+            const int buf = buffer(j);
+            wait_soon(&b->s_full[buf], phase(j), abort_flag, p.status, 39, p.wait_ns);
             tc_fence_after();
             uint32_t s[2][32];
             tmem_ld32(tmem + buf * kTile + lanes, s[0]);
@@ -311,7 +328,7 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
             if (it == 0) {
                 m = top;
             } else if (__any_sync(0xffffffffu, top > m + 8.f)) {
-                wait_soon(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 40, p.wait_ns);
+                wait_soon(&b->o_done[buffer(j - 2)], phase(j - 2), abort_flag, p.status, 40, p.wait_ns);
                 const float m_new = fmaxf(m, top), f = m_new == -INFINITY ? 1.f : exp2f(m - m_new);
                 tc_fence_after();
 #pragma unroll 1
@@ -346,7 +363,10 @@ __global__ void __launch_bounds__(kThreadsP, 1) latent_prefill_kernel(const __gr
             tc_fence_before();
             mbar_arrive(&b->p_full[buf]);
         }
-        if (it > 0) mbar_wait(&b->o_done[g], (it - 1) & 1u, abort_flag, p.status, 41, p.wait_ns);
+        if (it > 0) {
+            const int last = g + 2 * (it - 1);
+            mbar_wait(&b->o_done[buffer(last)], phase(last), abort_flag, p.status, 41, p.wait_ns);
+        }
         stat[g * kRows + r] = m;
         stat[(2 + g) * kRows + r] = l;
         tc_fence_before();
