@@ -1,7 +1,8 @@
 // Runner of the config-driven decoder (tlc_decoder_* of include/tlcuda.h): dense bf16 or f32
 // weights, layers described one by one.
 //
-// Two forms of the same layers:
+// Layers over several residual streams are in tlc_decoder_streams.cu.  Layers with one residual come in
+// two forms:
 //   one row (a decode step, a portion of one token), three launches per layer, four with experts:
 //     [norms + q, k, gate/up (or shared gate/up, router, shared gate)]
 //     [q/k norm + rotation + cache append + windowed attention]

@@ -661,9 +661,9 @@ template <typename T>
 int32_t launch_latent_query(tlc_ctx *ctx, const LatentParams &p) {
     constexpr int N = Vec<T>::N;
     const int DR = p.D + p.R, qpieces = (p.QR + N - 1) / N;
-    // CTAs per head: enough for the SMs, at most eight (a portable cluster), no more than pieces of the latent
+    // CTAs per head: up to two per SM, at most eight (a portable cluster), no more than pieces of the latent
     int C = 1;
-    while (C < 8 && (long)2 * C * (p.H + 1) * p.m <= ctx->sm_count && 2 * C <= p.kp / N) C *= 2;
+    while (C < 8 && (long)C * (p.H + 1) * p.m <= ctx->sm_count && 2 * C <= p.kp / N) C *= 2;
     const int split = (qpieces + 32 * kBatch - 1) / (32 * kBatch);  // stretches a row of W_uq is cut into
     const size_t area = std::max((size_t)kQueryThreads * N, p.q ? 0 : (size_t)((DR + C - 1) / C) * split);
     const size_t smem = ((size_t)((DR + 3) & ~3) + (p.q ? 0 : (size_t)qpieces * N) + area) * sizeof(float);
